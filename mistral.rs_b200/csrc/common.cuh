@@ -2,7 +2,7 @@
 //
 // Block layouts follow the ggml formats the reference consumes
 // (REF: mistralrs-quant/kernels/mmvq_gguf/mmvq_gguf.cu:134-225).  Everything here is
-// written for sm_100a only: mbarrier + cp.async.bulk (TMA engine, SASS UBLKCP), PDL
+// written for sm_100a only: mbarrier + cp.async.bulk (TMA engine), PDL
 // (griddepcontrol), 32-wide shuffles.
 #pragma once
 #include <cuda_bf16.h>
@@ -157,8 +157,8 @@ __device__ __forceinline__ void pdl_launch_dependents() {
 }
 
 // explicit shared-space accesses through 32-bit shared addresses: a pointer derived from a kernel's dynamic
-// shared memory by byte arithmetic is "generic" to the compiler (SASS LD.E / ST.E with an address-space
-// check, accounted as long-scoreboard traffic); these force LDS / STS
+// shared memory by byte arithmetic is a generic address to the compiler, and accesses through it are
+// accounted as long-scoreboard stalls; these name the shared state space
 __device__ __forceinline__ uint4 lds128(uint32_t saddr) {
   uint4 v;
   asm volatile("ld.shared.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(saddr));

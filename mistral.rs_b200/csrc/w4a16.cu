@@ -391,8 +391,7 @@ w4a16_int4_kernel(const __grid_constant__ CUtensorMap tmap_x, const WaParams p) 
   if (warp == 0) {
     // ===================== raw producer: the HBM stream =====================
     // The whole warp runs this loop convergently with warp-uniform operands; one elected lane issues each copy
-    // (inside an `if (lane == 0)` region every UBLKCP sits in an ELECT ... BRA.U.ANY loop and the address
-    // arithmetic runs through R2UR waterfalls: ~300 clocks per copy measured — the producer paced the kernel).
+    // (inside an `if (lane == 0)` region ~300 clocks per copy were measured — the producer paced the kernel).
     // Per iteration: the packed nibbles of one or two 64-k chunks, plus the scale row (and AWQ zero-point row) of
     // every group the iteration's k range touches (one row when group % 128 == 0) — the dequantisers read them
     // from the stage with LDS; nothing on their path waits for global memory.
