@@ -80,6 +80,9 @@ int mrs_seq_embed_pair(const void *table, const void *pairs, int dtype, const in
  *                                                    an entry may be dst, which then already holds this token's v)
  *   mixed[t] = v
  *   next_out[t] = v / sqrt(mean(v^2) + eps) * next_w   (the next sublayer's input, activation type)
+ * center != 0: a layer norm instead, next_out[t] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * next_w + next_b (next_b NULL: no
+ * bias; it is added in the RMS form too).  rows (NULL: all tokens in order; needs dst, y, hist and mixed NULL): output row t
+ * is formed from src[rows[t]].
  * With hist = the embedding output followed by every layer's result so far this is the depth-weighted average of
  * DenseFormer-style models; without it, the plain pre-norm residual step with a multiplier. */
 typedef struct {
@@ -98,6 +101,9 @@ typedef struct {
   int dtype, n_tok, width;
   const float *post_w;
   const float *add_vec;
+  const float *next_b;
+  int center;
+  const int32_t *rows;
 } mrs_seq_rms_residual_args;
 int mrs_seq_rms_residual(const mrs_seq_rms_residual_args *args, int64_t stream);
 
@@ -116,6 +122,8 @@ int mrs_seq_bounded_gate(const void *raw, int64_t raw_ld, int dtype, const float
  * logarithm is a softened log-sigmoid (power = 1 / temperature). */
 int mrs_seq_power_gate(const void *raw, int64_t raw_ld, int dtype, const float *bias, float power, int n_tok, int cols, float *gate,
                        int64_t stream);
+/* out[i] = cap * tanh(scale * x[i] / cap) in f32 (cap <= 0: scale * x[i]): logits with a multiplier and a soft cap. */
+int mrs_seq_soft_cap(const void *x, int dtype, float scale, float cap, int64_t n, float *out, int64_t stream);
 /* Root-mean-square norm of f32 rows in `groups` equal parts, times weight, with a gate read from an activation
  * tensor (row stride gate_ld): gate_first != 0: norm(x * act(gate)) * w; else norm(x) * w * act(gate).  The result,
  * times out_scale, goes to out[t * out_ld + c]. */
@@ -204,9 +212,12 @@ int mrs_seq_window_attention(const void *q, int64_t q_ld, const void *k_cache, c
 /* The general forms of the two calls above.
  * prepare: norm_mode 0 none, 1 per head (weights [dk], shared by the heads), 2 over the whole projection at once
  * (weights [heads * dk] and [kv_heads * dk]); then rotation of the first rot_dims entries of every q / k head in pairs
- * (i, i + rot_dims / 2) by cos_sin f32 [n_tok, rot_dims / 2, 2] (NULL: none); q and k change in place, k and v go to their
- * cache slots.  v NULL: the values are the keys as projected (before norm and rotation; needs dv == dk). */
+ * (`pairing`: i with i + rot_dims / 2, or neighbours 2 i and 2 i + 1) by cos_sin f32 [n_tok, rot_dims / 2, 2] (NULL: none); q and
+ * k change in place, k and v go to their cache slots.  v NULL: the values are the keys as projected (before norm and rotation;
+ * needs dv == dk). */
 enum { MRS_SEQ_QK_NORM_NONE = 0, MRS_SEQ_QK_NORM_HEAD = 1, MRS_SEQ_QK_NORM_WHOLE = 2 };
+/* which two entries make rotated pair i of n: (i, i + n) or (2 i, 2 i + 1) */
+enum { MRS_SEQ_PAIRS_HALVES = 0, MRS_SEQ_PAIRS_NEIGHBOURS = 1 };
 typedef struct {
   void *q, *k;
   const void *v;
@@ -220,6 +231,7 @@ typedef struct {
   void *k_cache, *v_cache;
   const int64_t *slot_of_tok;
   int n_tok;
+  int pairing;
 } mrs_seq_attn_prepare_args;
 int mrs_seq_attention_prepare(const mrs_seq_attn_prepare_args *args, int64_t stream);
 /* cos_sin[t][i] = mag * (cos, sin)(pos_of_tok[t] * freq[i]), i < half; the angle and its cos / sin in double. */
@@ -253,6 +265,8 @@ typedef struct {
   int out_f32;            /* != 0: out is f32 whatever the activation type */
   int64_t out_head;       /* elements between the heads of an output row; 0: dv.  With v_shared, a call may cover a column range of
                              the value heads (v_cache advanced to it) and write the same range of every head's output */
+  int chunk;              /* > 0: position i sees j only in its own chunk, floor(i / chunk) == floor(j / chunk), chunks counted from
+                             position 0 of the sequence (combines with window; keep_first and pool must be 0) */
 } mrs_seq_paged_attention_args;
 int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args, int64_t stream);
 /* Averaged cache entries for attention over pooled blocks: for every token of the step whose position ends a block of `pool`
@@ -285,12 +299,31 @@ int mrs_seq_prompt_attention_pooled(const void *q, int64_t q_ld, const void *k_c
                                     const int32_t *portions, int n_portions, int longest, const int32_t *pages, int pages_ld,
                                     int page_size, int heads, int kv_heads, int d, float scale, int window, int keep_first,
                                     const float *sink, int pool, int64_t pool_base, int every_value_head, int64_t stream);
+/* The same with every choice in one structure, and with chunks (as in mrs_seq_paged_attention_args). */
+typedef struct {
+  const void *q;
+  int64_t q_ld;
+  const void *k_cache, *v_cache;
+  void *out;
+  int64_t out_ld;
+  const int32_t *portions;
+  int n_portions, longest;
+  const int32_t *pages;
+  int pages_ld, page_size, heads, kv_heads, d;
+  float scale;
+  int window, keep_first;
+  const float *sink;
+  int pool;
+  int64_t pool_base;
+  int every_value_head, chunk;
+} mrs_seq_prompt_attention_args;
+int mrs_seq_prompt_attention_general(const mrs_seq_prompt_attention_args *args, int64_t stream);
 /* ---- attention through a shared latent ----------------------------------------------------------------- */
 /* Per token, from the columns of one projection y (row stride y_ld, activation type), any part optional:
  *   q_out[t] = rms_norm(y[t][q_col : q_col + q_rank]) * q_norm_w                      (the query latent, activation type)
  *   cache[slot(t)][0 : kv_rank] = rms_norm(y[t][kv_col : kv_col + kv_rank]) * kv_norm_w   (the key/value latent)
  *   cache[slot(t)][kv_rank : kv_rank + rot_dim] = turn(y[t][kv_col + kv_rank : ...])     (the key part all heads share)
- * turn: entries (2i, 2i + 1), i < rot_dims / 2, rotate by cos_sin[t][i] (f32 [n_tok, rot_dims / 2, 2]); the rest pass.
+ * turn: pair i < rot_dims / 2 (`pairing`) rotates by cos_sin[t][i] (f32 [n_tok, rot_dims / 2, 2]); the rest pass.
  * cache rows are cache_row elements apart.  q_rank 0: no query part; kv_rank 0: no cache part.  kv_out (optional): the normed
  * key/value latent also goes to kv_out[t][0 : kv_rank] (row stride kv_out_ld), for callers that decompress keys and values
  * of the step's own tokens with a matrix product. */
@@ -312,12 +345,16 @@ typedef struct {
   int n_tok;
   void *kv_out;
   int64_t kv_out_ld;
+  int pairing;
 } mrs_seq_latent_prepare_args;
 int mrs_seq_latent_prepare(const mrs_seq_latent_prepare_args *args, int64_t stream);
 /* out[t][h][0:dims] = in[t][h][0:dims] with entries (2i, 2i + 1), i < rot_dims / 2, rotated by cos_sin[t][i], the rest
  * copied.  in / out: activation type, row strides in_ld / out_ld, head strides in_head / out_head (elements). */
 int mrs_seq_rotate_pairs(const void *in, int64_t in_ld, int64_t in_head, void *out, int64_t out_ld, int64_t out_head, int dtype,
                          int heads, int dims, int rot_dims, const float *cos_sin, int n_tok, int64_t stream);
+/* the same with the pairing open (MRS_SEQ_PAIRS_*) */
+int mrs_seq_rotate_heads(const void *in, int64_t in_ld, int64_t in_head, void *out, int64_t out_ld, int64_t out_head, int dtype,
+                         int heads, int dims, int rot_dims, int pairing, const float *cos_sin, int n_tok, int64_t stream);
 
 /* The long portions of a step on tensor cores, in the absorbed form: q [n_tok, heads, kv_rank + rot_dim] (row stride q_ld) holds
  * per head [W_uk^T q_plain | q_rot]; the cached rows (cache_row elements apart) are at once the keys (all kv_rank + rot_dim

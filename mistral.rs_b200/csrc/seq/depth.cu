@@ -1,4 +1,4 @@
-// depth.cu — a single f32 residual with RMS norms whose sublayer outputs are added with a multiplier and whose layers
+// depth.cu — a single f32 residual with RMS norms (or layer norms with a bias) whose sublayer outputs are added with a multiplier and whose layers
 // hand on a depth-weighted average: what enters layer i + 1 is a learned mix of the embedding output and the results of
 // layers 0 .. i (the averaging of DenseFormer-style models), not layer i's result alone.  One kernel per sublayer does
 // the residual add, stores the layer's result into the step's history, forms the mix over the history and produces the
@@ -46,7 +46,7 @@ __global__ void __launch_bounds__(1024) rms_residual_kernel(const mrs_seq_rms_re
   __shared__ float red[33];
   __shared__ float mix[128];
   const int t = blockIdx.x, width = a.width;
-  const int64_t at = (int64_t)t * width;
+  const int64_t at = (int64_t)t * width, src_at = a.rows ? (int64_t)a.rows[t] * width : at;
   const T *y = (const T *)a.y;
   const int n_hist = a.hist ? a.n_hist : 0;
   for (int j = threadIdx.x; j < n_hist; j += blockDim.x) mix[j] = a.mix[j];
@@ -69,8 +69,8 @@ __global__ void __launch_bounds__(1024) rms_residual_kernel(const mrs_seq_rms_re
   float ss = 0.0f;
   for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
     float v[VEC];
-    if (VEC == 4) { const float4 q = *(const float4 *)(a.src + at + c); v[0] = q.x; v[1 % VEC] = q.y; v[2 % VEC] = q.z; v[3 % VEC] = q.w; }
-    else v[0] = a.src[at + c];
+    if (VEC == 4) { const float4 q = *(const float4 *)(a.src + src_at + c); v[0] = q.x; v[1 % VEC] = q.y; v[2 % VEC] = q.z; v[3 % VEC] = q.w; }
+    else v[0] = a.src[src_at + c];
     if (y && a.post_w) {     // every thread re-reads the columns it staged itself
 #pragma unroll
       for (int e = 0; e < VEC; e++) v[e] = fmaf(a.mult, row[c + e] * inv_y * a.post_w[c + e], v[e]);
@@ -118,18 +118,34 @@ __global__ void __launch_bounds__(1024) rms_residual_kernel(const mrs_seq_rms_re
 #pragma unroll
     for (int e = 0; e < VEC; e++) {
       row[c + e] = v[e];
-      ss = fmaf(v[e], v[e], ss);
+      ss = a.center ? ss + v[e] : fmaf(v[e], v[e], ss);
     }
   }
   if (a.next_out == nullptr) return;
-  const float inv = rsqrtf_exact(block_sum(ss, red) / (float)width + a.eps);
+  ss = block_sum(ss, red) / (float)width;
+  float mean = 0.0f;
+  if (a.center) {          // layer norm: the mean first, then the squared deviations of the columns this thread staged
+    mean = ss;
+    ss = 0.0f;
+    for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+#pragma unroll
+      for (int e = 0; e < VEC; e++) {
+        const float dev = row[c + e] - mean;
+        row[c + e] = dev;
+        ss = fmaf(dev, dev, ss);
+      }
+    }
+    ss = block_sum(ss, red) / (float)width;
+  }
+  const float inv = rsqrtf_exact(ss + a.eps);
   T *out = (T *)a.next_out;
   for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {     // every thread re-reads the columns it wrote itself
     if (VEC == 4) {
-      const float4 w = *(const float4 *)(a.next_w + c);
-      store4<T>(out + at + c, make_float4(row[c] * inv * w.x, row[c + 1 % VEC] * inv * w.y, row[c + 2 % VEC] * inv * w.z, row[c + 3 % VEC] * inv * w.w));
+      const float4 w = *(const float4 *)(a.next_w + c), b = a.next_b ? *(const float4 *)(a.next_b + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      store4<T>(out + at + c, make_float4(fmaf(row[c] * inv, w.x, b.x), fmaf(row[c + 1 % VEC] * inv, w.y, b.y),
+                                          fmaf(row[c + 2 % VEC] * inv, w.z, b.z), fmaf(row[c + 3 % VEC] * inv, w.w, b.w)));
     } else {
-      out[at + c] = from_f32<T>(row[c] * inv * a.next_w[c]);
+      out[at + c] = from_f32<T>(fmaf(row[c] * inv, a.next_w[c], a.next_b ? a.next_b[c] : 0.0f));
     }
   }
 }
@@ -158,15 +174,34 @@ extern "C" int mrs_seq_embed_pair(const void *table, const void *pairs, int dtyp
   return launch_status();
 }
 
+namespace seq {
+template <typename T>
+__global__ void soft_cap_kernel(const T *__restrict__ x, float scale, float cap, int64_t n, float *__restrict__ out) {
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const float z = to_f32<T>(x[i]) * scale;
+    out[i] = cap > 0.0f ? cap * tanhf(z / cap) : z;
+  }
+}
+}  // namespace seq
+
+extern "C" int mrs_seq_soft_cap(const void *x, int dtype, float scale, float cap, int64_t n, float *out, int64_t stream) {
+  if (n <= 0) return 0;
+  const int64_t blocks = (n + 255) / 256;
+  const int grid = (int)(blocks < 148 * 16 ? blocks : 148 * 16);
+  SEQ_DISPATCH_DTYPE(dtype, (soft_cap_kernel<T><<<grid, 256, 0, (cudaStream_t)stream>>>((const T *)x, scale, cap, n, out)));
+  return launch_status();
+}
+
 extern "C" int mrs_seq_rms_residual(const mrs_seq_rms_residual_args *args, int64_t stream) {
   const mrs_seq_rms_residual_args &a = *args;
   if (a.n_tok <= 0) return 0;
   if (!a.src || a.width <= 0 || (a.hist && (a.n_hist < 1 || a.n_hist > 128 || !a.mix)) || (a.next_out && !a.next_w)) return -2;
+  if (a.rows && (a.dst || a.y || a.hist || a.mixed)) return -2;
   const size_t bytes = (size_t)a.width * sizeof(float);
   if (bytes > 200 * 1024) return -2;
   auto al = [](const void *p) { return ((uintptr_t)p & 15) == 0; };
   const bool vec = a.width % 4 == 0 && al(a.src) && al(a.dst) && al(a.y) && al(a.hist) && a.hist_stride % 4 == 0 && al(a.mixed) &&
-                   al(a.next_w) && al(a.next_out);      // post_w and add_vec are read one element at a time
+                   al(a.next_w) && al(a.next_b) && al(a.next_out);      // post_w and add_vec are read one element at a time
   const int items = vec ? a.width / 4 : a.width;
   int th = 64;
   while (th < 1024 && th * (a.n_tok <= 64 ? 1 : 2) < items) th *= 2;    // short batches: one item per thread where possible

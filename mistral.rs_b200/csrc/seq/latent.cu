@@ -4,7 +4,8 @@
 // (W_uk,h^T q_h) . c + q_rot,h . k_rot and its output W_uv,h (sum_j p_j c_j): attention runs over the latent rows
 // themselves as ONE key/value head of size kv_rank + rot_dim whose values are the first kv_rank columns of the keys
 // (the paged kernels of window_attn.cu with row strides, or the tensor-core kernel of latent_attn_mma.cu).  This file
-// holds what surrounds the matrix products: the latent norms, the rotation in neighbouring pairs and the cache write.
+// holds what surrounds the matrix products: the latent norms, the rotation (in neighbouring pairs or in halves) and the
+// cache write.
 #include "seq_common.cuh"
 
 namespace seq {
@@ -49,34 +50,37 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const mrs_seq_laten
   src += a.kv_rank;
   dst += a.kv_rank;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const float u = to_f32<T>(src[2 * i]), v = to_f32<T>(src[2 * i + 1]);
+    const int iu = pair_u(i, a.pairing), iv = pair_v(i, half, a.pairing);
+    const float u = to_f32<T>(src[iu]), v = to_f32<T>(src[iv]);
     const float2 c = cs[i];
-    dst[2 * i] = from_f32<T>(u * c.x - v * c.y);
-    dst[2 * i + 1] = from_f32<T>(v * c.x + u * c.y);
+    dst[iu] = from_f32<T>(u * c.x - v * c.y);
+    dst[iv] = from_f32<T>(v * c.x + u * c.y);
   }
   for (int d = 2 * half + threadIdx.x; d < a.rot_dim; d += blockDim.x) dst[d] = src[d];
 }
 
-// one CTA per token, all heads: out[t][h][:dims] = in[t][h][:dims] with the first rot_dims entries turned in neighbouring pairs
+// one CTA per token, all heads: out[t][h][:dims] = in[t][h][:dims] with the first rot_dims entries turned in pairs.  In place
+// (out == in) is fine: a pair is read and written by one thread.
 template <typename T>
-__global__ void rotate_pairs_kernel(const T *__restrict__ in, int64_t in_ld, int64_t in_head, T *__restrict__ out, int64_t out_ld,
-                                    int64_t out_head, int heads, int dims, int rot_dims, const float2 *__restrict__ cos_sin) {
+__global__ void rotate_heads_kernel(const T *__restrict__ in, int64_t in_ld, int64_t in_head, T *__restrict__ out, int64_t out_ld,
+                                    int64_t out_head, int heads, int dims, int rot_dims, int pairing, const float2 *__restrict__ cos_sin) {
   const int t = blockIdx.x, half = cos_sin ? rot_dims / 2 : 0, pairs = dims / 2;
   const T *src = in + (int64_t)t * in_ld;
   T *dst = out + (int64_t)t * out_ld;
   const float2 *cs = cos_sin + (int64_t)t * half;
   for (int e = threadIdx.x; e < heads * pairs; e += blockDim.x) {
     const int h = e / pairs, i = e % pairs;
-    const T *s = src + (int64_t)h * in_head + 2 * i;
-    T *d = dst + (int64_t)h * out_head + 2 * i;
+    const T *s = src + (int64_t)h * in_head;
+    T *d = dst + (int64_t)h * out_head;
     if (i < half) {
-      const float u = to_f32<T>(s[0]), v = to_f32<T>(s[1]);
+      const int iu = pair_u(i, pairing), iv = pair_v(i, half, pairing);
+      const float u = to_f32<T>(s[iu]), v = to_f32<T>(s[iv]);
       const float2 c = cs[i];
-      d[0] = from_f32<T>(u * c.x - v * c.y);
-      d[1] = from_f32<T>(v * c.x + u * c.y);
-    } else {
-      d[0] = s[0];
-      d[1] = s[1];
+      d[iu] = from_f32<T>(u * c.x - v * c.y);
+      d[iv] = from_f32<T>(v * c.x + u * c.y);
+    } else {               // past the rotated entries: entries 2 i and 2 i + 1 pass
+      d[2 * i] = s[2 * i];
+      d[2 * i + 1] = s[2 * i + 1];
     }
   }
   if (dims & 1)
@@ -102,10 +106,17 @@ extern "C" int mrs_seq_latent_prepare(const mrs_seq_latent_prepare_args *args, i
 
 extern "C" int mrs_seq_rotate_pairs(const void *in, int64_t in_ld, int64_t in_head, void *out, int64_t out_ld, int64_t out_head, int dtype,
                                     int heads, int dims, int rot_dims, const float *cos_sin, int n_tok, int64_t stream) {
+  return mrs_seq_rotate_heads(in, in_ld, in_head, out, out_ld, out_head, dtype, heads, dims, rot_dims, MRS_SEQ_PAIRS_NEIGHBOURS, cos_sin, n_tok,
+                              stream);
+}
+
+extern "C" int mrs_seq_rotate_heads(const void *in, int64_t in_ld, int64_t in_head, void *out, int64_t out_ld, int64_t out_head, int dtype,
+                                    int heads, int dims, int rot_dims, int pairing, const float *cos_sin, int n_tok, int64_t stream) {
   if (n_tok <= 0 || heads <= 0 || dims <= 0) return 0;
   if (cos_sin && (rot_dims < 2 || rot_dims % 2 || rot_dims > dims)) return -2;
   const int items = heads * (dims / 2), th = items >= 256 ? 256 : (items >= 128 ? 128 : 64);
-  SEQ_DISPATCH_DTYPE(dtype, (rotate_pairs_kernel<T><<<n_tok, th, 0, (cudaStream_t)stream>>>(
-                                (const T *)in, in_ld, in_head, (T *)out, out_ld, out_head, heads, dims, rot_dims, (const float2 *)cos_sin)));
+  SEQ_DISPATCH_DTYPE(dtype, (rotate_heads_kernel<T><<<n_tok, th, 0, (cudaStream_t)stream>>>(
+                                (const T *)in, in_ld, in_head, (T *)out, out_ld, out_head, heads, dims, rot_dims, pairing,
+                                (const float2 *)cos_sin)));
   return launch_status();
 }

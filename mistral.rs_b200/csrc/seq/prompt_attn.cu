@@ -37,9 +37,17 @@ struct Params {
   const float *sink;
   int pool, per_page;          // pool > 0: averaged blocks before the window; per_page = ceil(page_size / pool)
   int64_t pool_base;
+  int chunk;                   // > 0: a query sees only keys of its own chunk of positions
   int v_heads;                 // 1, or the number of value heads when every head is applied to every value head
   int o_f32;                   // the result is f32 [tokens, heads, v_heads * D] (o is then float *)
 };
+
+// first position the query at `pos` sees through the window and / or its chunk (kept first positions aside)
+__device__ __forceinline__ int first_visible(const Params &p, int pos) {
+  int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  if (p.chunk > 0) lo = max(lo, pos - pos % p.chunk);
+  return lo;
+}
 
 template <int D>
 __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Params p) {
@@ -65,7 +73,8 @@ __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Para
 
   // key tiles of this query tile: the kept first positions that lie before the window's first tile, then the window
   const int kv_end = min(total, past + q0 + BM);
-  const int win_begin = p.window > 0 ? max(0, past + q0 - p.window + 1) / BN * BN : 0;
+  const int first_key = first_visible(p, past + q0);                 // of the tile's first query; later queries start no earlier
+  const int win_begin = first_key / BN * BN;
   // entries before the window: kept first positions, or averaged blocks (as many as the tile's last query sees)
   const int kept_end = p.pool > 0 ? max(0, kv_end - p.window) / p.pool : min(p.keep_first, win_begin);
   const int kept_tiles = (kept_end + BN - 1) / BN;                  // kept_tiles * BN <= win_begin: no key twice
@@ -116,6 +125,8 @@ __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Para
   for (int i = 0; i < DT; i++) { oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f; }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int row_a = q0 + warp * 16 + (lane >> 2);   // this thread's accumulator rows (inside the portion): row_a, row_a + 8
+  const int lo_row[2] = {first_visible(p, past + row_a), first_visible(p, past + row_a + 8)};
+  const int warp_first = past + q0 + warp * 16, warp_lo = first_visible(p, warp_first), warp_lo_last = first_visible(p, warp_first + 15);
 
   for (int t = 0; t < nt; t++) {
     const int buf = t & 1;
@@ -124,6 +135,11 @@ __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Para
     cp_async_wait<1>();
     __syncthreads();
     const int t0 = tile_start(t);
+    // a tile that none of this warp's rows sees (above its diagonal, or wholly before its window or chunk) is not computed
+    if (t >= kept_tiles && (t0 > warp_first + 15 || (t0 + BN <= warp_lo && p.keep_first <= t0))) {
+      __syncthreads();
+      continue;
+    }
 
     float sacc[BN / 8][4];
 #pragma unroll
@@ -141,7 +157,7 @@ __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Para
       }
     }
 
-    const bool need_mask = p.window > 0 || t0 + BN > kv_end || t0 + BN - 1 > past + q0 + warp * 16;
+    const bool need_mask = t < kept_tiles || t0 < warp_lo_last || t0 + BN > kv_end || t0 + BN - 1 > warp_first;
     float mx[2] = {m_run[0], m_run[1]};
 #pragma unroll
     for (int j = 0; j < BN / 8; j++) {
@@ -153,7 +169,7 @@ __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Para
           const int row = past + row_a + ((e >> 1) << 3);          // the query's position
           bool ok;
           if (p.pool > 0 && t < kept_tiles) ok = (col + 1) * p.pool - 1 <= row - p.window;        // the block ends at or before row - window
-          else ok = col < total && col <= row && (p.window <= 0 || row - col < p.window || col < p.keep_first);
+          else ok = col < total && col <= row && (col >= lo_row[e >> 1] || col < p.keep_first);
           if (!ok) s = -INFINITY;
         }
         sacc[j][e] = s;
@@ -248,24 +264,39 @@ extern "C" int mrs_seq_prompt_attention(const void *q, int64_t q_ld, const void 
                                          kv_heads, d, scale, window, keep_first, sink, 0, 0, 0, stream);
 }
 
+extern "C" int mrs_seq_prompt_attention_general(const mrs_seq_prompt_attention_args *args, int64_t stream) {
+  const mrs_seq_prompt_attention_args &a = *args;
+  const int heads = a.heads, kv_heads = a.kv_heads, d = a.d, pool = a.pool > 0 ? a.pool : 0, chunk = a.chunk > 0 ? a.chunk : 0;
+  if (a.n_portions <= 0 || a.longest <= 0) return 0;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || (d != 64 && d != 128) || !a.portions || !a.pages || a.page_size <= 0) return -2;
+  if (pool > 0 && (a.window <= 0 || a.keep_first > 0)) return -2;
+  if (chunk > 0 && (a.keep_first > 0 || pool > 0)) return -2;
+  if ((int64_t)heads * (a.every_value_head ? kv_heads : 1) > 65535) return -2;
+  if ((a.q_ld | a.out_ld) % 8 || (((uintptr_t)a.q | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache | (uintptr_t)a.out) & 15)) return -3;
+  seqp::Params p = {};
+  p.q = (const __nv_bfloat16 *)a.q; p.k_cache = (const __nv_bfloat16 *)a.k_cache; p.v_cache = (const __nv_bfloat16 *)a.v_cache;
+  p.o = (__nv_bfloat16 *)a.out;
+  p.portions = a.portions; p.pages = a.pages; p.pages_ld = a.pages_ld; p.page_size = a.page_size;
+  p.H = heads; p.KVH = kv_heads; p.q_ld = a.q_ld; p.o_ld = a.out_ld;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.window = a.window; p.keep_first = a.keep_first > 0 ? a.keep_first : 0; p.sink = a.sink;
+  p.pool = pool; p.per_page = pool > 0 ? (a.page_size + pool - 1) / pool : 0; p.pool_base = a.pool_base;
+  p.chunk = chunk;
+  p.v_heads = a.every_value_head ? kv_heads : 1;
+  p.o_f32 = a.every_value_head ? 1 : 0;
+  return d == 128 ? seqp::launch<128>(p, a.n_portions, a.longest, (cudaStream_t)stream)
+                  : seqp::launch<64>(p, a.n_portions, a.longest, (cudaStream_t)stream);
+}
+
 extern "C" int mrs_seq_prompt_attention_pooled(const void *q, int64_t q_ld, const void *k_cache, const void *v_cache, void *out, int64_t out_ld,
                                                const int32_t *portions, int n_portions, int longest, const int32_t *pages, int pages_ld,
                                                int page_size, int heads, int kv_heads, int d, float scale, int window, int keep_first,
                                                const float *sink, int pool, int64_t pool_base, int every_value_head, int64_t stream) {
-  if (n_portions <= 0 || longest <= 0) return 0;
-  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || (d != 64 && d != 128) || !portions || !pages || page_size <= 0) return -2;
-  if (pool > 0 && (window <= 0 || keep_first > 0)) return -2;
-  if ((int64_t)heads * (every_value_head ? kv_heads : 1) > 65535) return -2;
-  if ((q_ld | out_ld) % 8 || (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15)) return -3;
-  seqp::Params p = {};
-  p.q = (const __nv_bfloat16 *)q; p.k_cache = (const __nv_bfloat16 *)k_cache; p.v_cache = (const __nv_bfloat16 *)v_cache;
-  p.o = (__nv_bfloat16 *)out;
-  p.portions = portions; p.pages = pages; p.pages_ld = pages_ld; p.page_size = page_size;
-  p.H = heads; p.KVH = kv_heads; p.q_ld = q_ld; p.o_ld = out_ld;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window; p.keep_first = keep_first > 0 ? keep_first : 0; p.sink = sink;
-  p.pool = pool > 0 ? pool : 0; p.per_page = pool > 0 ? (page_size + pool - 1) / pool : 0; p.pool_base = pool_base;
-  p.v_heads = every_value_head ? kv_heads : 1;
-  p.o_f32 = every_value_head ? 1 : 0;
-  return d == 128 ? seqp::launch<128>(p, n_portions, longest, (cudaStream_t)stream) : seqp::launch<64>(p, n_portions, longest, (cudaStream_t)stream);
+  mrs_seq_prompt_attention_args a = {};
+  a.q = q; a.q_ld = q_ld; a.k_cache = k_cache; a.v_cache = v_cache; a.out = out; a.out_ld = out_ld;
+  a.portions = portions; a.n_portions = n_portions; a.longest = longest;
+  a.pages = pages; a.pages_ld = pages_ld; a.page_size = page_size; a.heads = heads; a.kv_heads = kv_heads; a.d = d;
+  a.scale = scale; a.window = window; a.keep_first = keep_first; a.sink = sink;
+  a.pool = pool; a.pool_base = pool_base; a.every_value_head = every_value_head;
+  return mrs_seq_prompt_attention_general(&a, stream);
 }

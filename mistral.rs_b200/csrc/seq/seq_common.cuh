@@ -50,6 +50,10 @@ __device__ __forceinline__ float glu_join(float g, float u, const mrs_seq_glu_ru
   return apply_act(g, r.act) * u;
 }
 
+// ---- the two entries of rotated pair i of n (MRS_SEQ_PAIRS_*) ----------------------------------------
+__device__ __forceinline__ int pair_u(int i, int pairing) { return pairing == MRS_SEQ_PAIRS_NEIGHBOURS ? 2 * i : i; }
+__device__ __forceinline__ int pair_v(int i, int n, int pairing) { return pairing == MRS_SEQ_PAIRS_NEIGHBOURS ? 2 * i + 1 : i + n; }
+
 // ---- reductions -------------------------------------------------------------------------------------
 __device__ __forceinline__ float warp_sum(float x) {
 #pragma unroll

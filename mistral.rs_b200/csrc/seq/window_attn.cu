@@ -1,6 +1,6 @@
 // window_attn.cu — softmax attention over a paged cache: RMS norm of queries and keys (per head, or over the whole
 // projection), optional rotary positions on part of every head, a sliding window (or full causal reach) that may keep
-// the first tokens of the sequence in sight, an optional per-head sink in the softmax denominator, grouped key/value
+// the first tokens of the sequence in sight, or chunks of the sequence that see only themselves, an optional per-head sink in the softmax denominator, grouped key/value
 // heads, values that may be the unnormed keys, and key / value head sizes that need not match.  The new tokens' keys and values are stored first; the attention kernel then reads
 // every key of a query, old or new, from the pages — one code path for a prompt portion and for a decoded token.
 #include "seq_common.cuh"
@@ -9,7 +9,7 @@ namespace seq {
 
 // Query / key preparation, one CTA per token.  Phase 1: sums of squares per head (one warp per q or k head).  Phase 2,
 // again one warp per head: the RMS norm (per head with weights shared by the heads, or over the whole projection at
-// once with one weight per element), the rotation of the first rot_dims entries in pairs (i, i + rot_dims / 2) by the
+// once with one weight per element), the rotation of the first rot_dims entries in pairs (halves or neighbours) by the
 // step's cos / sin table, q and k rewritten in place, k stored to its cache slot; values stored from their own
 // projection or — v == NULL — from the keys as they were projected (read before the key is rewritten).
 template <typename T>
@@ -61,13 +61,14 @@ __global__ void attention_prepare_kernel(const mrs_seq_attn_prepare_args a) {
         __syncwarp();
       }
       for (int i = lane; i < half; i += 32) {          // rotated pairs
-        const float u = normed ? to_f32<T>(src[i]) * inv * w[i] : to_f32<T>(src[i]);
-        const float v = normed ? to_f32<T>(src[i + half]) * inv * w[i + half] : to_f32<T>(src[i + half]);
+        const int iu = pair_u(i, a.pairing), iv = pair_v(i, half, a.pairing);
+        const float u = normed ? to_f32<T>(src[iu]) * inv * w[iu] : to_f32<T>(src[iu]);
+        const float v = normed ? to_f32<T>(src[iv]) * inv * w[iv] : to_f32<T>(src[iv]);
         const float2 c = cs[i];
         const T ru = from_f32<T>(u * c.x - v * c.y), rv = from_f32<T>(v * c.x + u * c.y);
-        src[i] = ru;
-        src[i + half] = rv;
-        if (cached) { cached[i] = ru; cached[i + half] = rv; }
+        src[iu] = ru;
+        src[iv] = rv;
+        if (cached) { cached[iu] = ru; cached[iv] = rv; }
       }
       for (int d = 2 * half + lane; d < dk; d += 32) {  // the rest passes
         const T r = normed ? from_f32<T>(to_f32<T>(src[d]) * inv * w[d]) : src[d];
@@ -103,6 +104,12 @@ __device__ __forceinline__ int64_t key_row(const int32_t *table, int j, int pool
   const int page = (j * pool) / page_size, first = (page * page_size + pool - 1) / pool;
   return pool_base + (int64_t)table[page] * per_page + (j - first);
 }
+// First position a query sees through a sliding window and / or through chunks counted from position 0
+__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
+  int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  if (chunk > 0) lo = max(lo, pos - pos % chunk);
+  return lo;
+}
 template <typename T> __device__ __forceinline__ void store_out(T *out, int64_t at, float v, int as_f32) {
   if (as_f32) ((float *)out)[at] = v;
   else out[at] = from_f32<T>(v);
@@ -119,7 +126,8 @@ __global__ void __launch_bounds__(128) window_attention_kernel(const T *__restri
                                                                int pages_ld, int page_size, const int32_t *__restrict__ seq_of_tok,
                                                                const int32_t *__restrict__ pos_of_tok, const int32_t *__restrict__ tok_index,
                                                                int n_tok, T *__restrict__ out, int64_t out_ld, float out_scale, int64_t k_row,
-                                                               int64_t v_row, int pool, int64_t pool_base, int v_shared, int out_f32, int64_t out_head) {
+                                                               int64_t v_row, int pool, int64_t pool_base, int v_shared, int out_f32, int64_t out_head,
+    int chunk) {
   extern __shared__ __align__(16) float qsm[];   // [warps][dk]
   const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
   const int64_t job = (int64_t)blockIdx.x * (blockDim.x >> 5) + wib;
@@ -130,7 +138,7 @@ __global__ void __launch_bounds__(128) window_attention_kernel(const T *__restri
   for (int d = lane; d < dk; d += 32) qv[d] = to_f32<T>(q[(int64_t)t * q_ld + h * dk + d]) * scale;
   __syncwarp();
   const int32_t *table = pages + (int64_t)s * pages_ld;
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int lo = first_visible(pos, window, chunk);
   float m = -INFINITY, l = 0.0f, acc[MAX_VCOLS];
 #pragma unroll
   for (int c = 0; c < MAX_VCOLS; c++) acc[c] = 0.0f;
@@ -188,7 +196,8 @@ __global__ void __launch_bounds__(SPLIT * 32) window_attention_vec_kernel(
     const T *__restrict__ q, int64_t q_ld, const T *__restrict__ k_cache, const T *__restrict__ v_cache, int heads, int kv_heads, int dk, int dv,
     float scale, int window, int keep_first, const float *__restrict__ sink, const int32_t *__restrict__ pages, int pages_ld, int page_size,
     const int32_t *__restrict__ seq_of_tok, const int32_t *__restrict__ pos_of_tok, const int32_t *__restrict__ tok_index, T *__restrict__ out,
-    int64_t out_ld, float out_scale, int64_t k_row, int64_t v_row, int pool, int64_t pool_base, int v_shared, int out_f32, int64_t out_head) {
+    int64_t out_ld, float out_scale, int64_t k_row, int64_t v_row, int pool, int64_t pool_base, int v_shared, int out_f32, int64_t out_head,
+    int chunk) {
   extern __shared__ __align__(16) float sm[];   // q [dk] | per warp: m, l, acc [VPAIRS * 64]
   const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
   const int ti = blockIdx.x / heads, h = blockIdx.x % heads, t = tok_index ? tok_index[ti] : ti, g = h / (heads / kv_heads);
@@ -197,7 +206,7 @@ __global__ void __launch_bounds__(SPLIT * 32) window_attention_vec_kernel(
   for (int d = threadIdx.x; d < dk; d += SPLIT * 32) qv[d] = to_f32<T>(q[(int64_t)t * q_ld + h * dk + d]) * scale;
   __syncthreads();
   const int32_t *table = pages + (int64_t)s * pages_ld;
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int lo = first_visible(pos, window, chunk);
   float m = -INFINITY, l = 0.0f;
   float2 acc[VPAIRS];
 #pragma unroll
@@ -334,6 +343,8 @@ extern "C" int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args,
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || dv > 1024 || dk > 2048 || a.page_size <= 0) return -2;
   const int keep_first = a.keep_first > 0 ? a.keep_first : 0, pool = a.pool > 0 ? a.pool : 0;
   if (pool > 0 && (a.window <= 0 || keep_first > 0)) return -2;      // averaged blocks lie before a window and replace kept first keys
+  const int chunk = a.chunk > 0 ? a.chunk : 0;
+  if (chunk > 0 && (keep_first > 0 || pool > 0)) return -2;          // what lies before the chunk is not seen
   cudaStream_t st = (cudaStream_t)stream;
   const int elem = dtype == MRS_SEQ_BF16 ? 2 : 4;
   const int64_t k_row = a.k_row > 0 ? a.k_row : (int64_t)kv_heads * dk, v_row = a.v_row > 0 ? a.v_row : (int64_t)kv_heads * dv;
@@ -346,7 +357,7 @@ extern "C" int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args,
   window_attention_vec_kernel<T, VP, SPLIT><<<(unsigned)n_tok * heads, SPLIT * 32, (dk + SPLIT * (2 + VP * 64)) * sizeof(float), st>>>( \
       (const T *)a.q, a.q_ld, (const T *)a.k_cache, (const T *)a.v_cache, heads, kv_heads, dk, dv, a.scale, a.window, keep_first, a.sink,  \
       a.pages, a.pages_ld, a.page_size, a.seq_of_tok, a.pos_of_tok, a.tok_index, (T *)a.out, a.out_ld, a.out_scale, k_row, v_row, pool,     \
-      a.pool_base, a.v_shared, a.out_f32, out_head)
+      a.pool_base, a.v_shared, a.out_f32, out_head, chunk)
     SEQ_DISPATCH_DTYPE(dtype, {
       if (dv <= 64) SEQ_ATTN_VEC(1);
       else if (dv <= 128) SEQ_ATTN_VEC(2);
@@ -362,7 +373,7 @@ extern "C" int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args,
   window_attention_kernel<T, VC><<<(unsigned)((jobs + warps - 1) / warps), warps * 32, warps * dk * sizeof(float), st>>>(  \
       (const T *)a.q, a.q_ld, (const T *)a.k_cache, (const T *)a.v_cache, heads, kv_heads, dk, dv, a.scale, a.window, keep_first, a.sink, \
       a.pages, a.pages_ld, a.page_size, a.seq_of_tok, a.pos_of_tok, a.tok_index, n_tok, (T *)a.out, a.out_ld, a.out_scale, k_row, v_row, pool, \
-      a.pool_base, a.v_shared, a.out_f32, out_head)
+      a.pool_base, a.v_shared, a.out_f32, out_head, chunk)
   SEQ_DISPATCH_DTYPE(dtype, {
     if (dv <= 64) SEQ_ATTN_LAUNCH(2);
     else if (dv <= 128) SEQ_ATTN_LAUNCH(4);

@@ -7,8 +7,9 @@ layer may reuse), a linear recurrence whose per-channel forget gate also writes 
 to a sublayer's input, a Mamba-2 style state-space mixer, two mixers side by side, dense GLU / plain and routed-expert
 feed-forwards (softmax or sigmoid routing, groups scored by their best or their few best experts, plain or capped GLU),
 a token shift (a sublayer's input blended with its predecessor's), gated linear attention with a decay per key channel,
-attention whose far past is seen as averaged blocks and whose softmax weights are mixed across heads, output gates per
-entry or per head.
+attention whose far past is seen as averaged blocks and whose softmax weights are mixed across heads, attention inside
+chunks of the sequence, output gates per entry or per head, layer norms around a single residual, logits with a multiplier
+and a soft cap.
 
 A mechanism owns its device weights and declares the per-layer cache it needs (`alloc_cache`): token-indexed pages
 (sized by the engine's block pool) and / or per-request state slots (sized by the engine's slot pool).  `forward`
@@ -61,6 +62,21 @@ class TanhNorm:
         self.t = (alpha, weight, bias)
 
 
+class LayerNorm:
+    """(x - mean) / sqrt(mean squared deviation + eps) * weight + bias, in f32, fused with the residual add before it:
+    `after_add` is x += y (y: a sublayer's output) followed by the norm, in one pass over the f32 residual x [T, W]."""
+
+    def __init__(self, weight, bias, eps):
+        self.weight, self.bias, self.eps = weight, bias, eps
+
+    def of(self, x, dtype, rows=None):
+        """The norm of x, or of its rows `rows` only."""
+        return K.rms_residual(x, next_w=self.weight, next_b=self.bias, center=True, eps=self.eps, dtype=dtype, rows=rows)
+
+    def after_add(self, x, y):
+        return K.rms_residual(x, y, dst=x, next_w=self.weight, next_b=self.bias, center=True, eps=self.eps)
+
+
 class Rotation:
     """Rotary positions on the first `dims` entries of every head, frequency base^(-2i/dims) for pair i.  Which two entries
     make pair i, (i, i + dims / 2) or the neighbours (2i, 2i + 1), is the choice of the kernel that applies the table.
@@ -111,8 +127,9 @@ class Rotation:
 class WindowAttention:
     """Grouped-query softmax attention over pages.  Queries and keys: RMS norm per head with weights shared by the
     heads (`norm_mode` QK_NORM_HEAD), over the whole projection at once (QK_NORM_WHOLE) or none; then `rotation` (None:
-    scores carry no position).  Scores are scaled by a given constant.  Position i sees j <= i with i - j < `window`
-    (0: full causal) or j < `keep_first`; `sink` [heads] adds exp(sink) to the softmax denominator.  With
+    scores carry no position; `pairing`: which two entries of a head turn together).  Scores are scaled by a given constant.
+    Position i sees j <= i with i - j < `window` (0: full causal) or j < `keep_first`; with `chunk` > 0 only positions of its own
+    chunk, floor(i / chunk) == floor(j / chunk), counted from position 0 of the sequence however its tokens come in; `sink` [heads] adds exp(sink) to the softmax denominator.  With
     `values_from_keys` there is no value projection: the values are the keys as projected, before norm and rotation.
 
     `pool` > 0 (needs a window and the page size): the positions before the window are seen block-wise — one key and one
@@ -125,10 +142,13 @@ class WindowAttention:
     attention kernel applies every head's weights to all value heads in f32, `seq_ops.mix_heads` sums over g."""
 
     def __init__(self, heads, kv_heads, dk, dv, scale, window, q_norm_w, k_norm_w, eps, norm_mode=K.QK_NORM_HEAD, rotation=None,
-                 keep_first=0, sink=None, values_from_keys=False, pool=0, talk=None, page_size=None):
+                 keep_first=0, sink=None, values_from_keys=False, pool=0, talk=None, page_size=None, chunk=0, pairing=K.PAIRS_HALVES):
         if pool > 0 and (window <= 0 or keep_first > 0 or not page_size):
             raise ValueError("averaged blocks need a window, no kept first tokens, and the page size")
+        if chunk > 0 and (pool > 0 or keep_first > 0):
+            raise ValueError("chunks hide everything before them: no averaged blocks, no kept first tokens")
         self.pool, self.talk, self.pool_page_size, self.pool_base = int(pool), talk, page_size, 0
+        self.chunk, self.pairing = int(chunk), pairing
         if values_from_keys and dk != dv:
             raise ValueError("values that are the keys need equal key and value head sizes")
         if heads % kv_heads:
@@ -150,7 +170,8 @@ class WindowAttention:
         return {"k": torch.zeros(rows, self.kv_heads, self.dk, dtype=dtype, device=device),
                 "v": torch.zeros(rows, self.kv_heads, self.dv, dtype=dtype, device=device)}
 
-    def attend(self, y, col0, batch, cache, page_size, out, out_col=0, out_scale=1.0, gate_col=None, gate_act=K.ACT_SIGMOID):
+    def attend(self, y, col0, batch, cache, page_size, out, out_col=0, out_scale=1.0, gate_col=None, gate_act=K.ACT_SIGMOID,
+               gate_group=1):
         """y holds q | k | v (q | k when the values are the keys) from column col0; writes heads * dv columns of `out`
         from out_col.  Keys and values of the new tokens are normed, rotated and stored first.  Long portions (32 tokens
         or more) run on tensor cores when they fit (bf16, equal head sizes of 64 or 128, 16-byte aligned rows): when every
@@ -158,30 +179,33 @@ class WindowAttention:
         kernels over the fresh q / k / v; otherwise — sinks, kept tokens, portions that continue a sequence — on the
         sequence library's prompt kernel, which reads keys and values from the pages.  Every other token (short portions,
         decoded tokens, other head sizes, f32) runs on the (token, head) kernel over the pages, and so does every token of a
-        layer with averaged blocks or mixed heads.  gate_col: columns of y (heads * dv of them) whose `gate_act` multiplies the
-        result entry by entry."""
+        layer with averaged blocks or mixed heads.  gate_col: columns of y whose `gate_act` multiplies the result, one column per
+        `gate_group` neighbouring entries (1: entry by entry; dv: one number per head, not with mixed heads)."""
         kc = col0 + self.heads * self.dk
         vc = None if self.values_from_keys else kc + self.kv_heads * self.dk
         cos_sin = self.rotation.table(batch) if self.rotation is not None else None
         K.attention_prepare(y, col0, kc, vc, self.norm_mode, self.q_norm_w, self.k_norm_w, self.eps, self.heads, self.kv_heads, self.dk,
-                            self.dv, cache["k"], cache["v"], batch.slot_of_tok, cos_sin, self.rotation.dims if cos_sin is not None else 0)
+                            self.dv, cache["k"], cache["v"], batch.slot_of_tok, cos_sin, self.rotation.dims if cos_sin is not None else 0,
+                            pairing=self.pairing)
         if self.pool > 0:
             if page_size != self.pool_page_size or cache["k"].shape[0] <= self.pool_base:
                 raise ValueError("the cache was not made for this layer's averaged blocks")
             K.pool_blocks(cache["k"], cache["v"], self.kv_heads * self.dk, self.kv_heads * self.dv, self.pool, self.pool_base, batch, page_size)
         if self.pool > 0 or self.talk is not None:
-            self._attend_general(y, col0, batch, cache, page_size, out, out_col, out_scale, gate_col, gate_act)
+            self._attend_general(y, col0, batch, cache, page_size, out, out_col, out_scale, gate_col, gate_act, gate_group)
             return
         self._attend_plain(y, col0, kc, vc, batch, cache, page_size, out, out_col, out_scale)
         if gate_col is not None:
-            K.gate_cols(out[:, out_col:], y, gate_col, self.heads * self.dv, 1, gate_act)
+            K.gate_cols(out[:, out_col:], y, gate_col, self.heads * self.dv, gate_group, gate_act)
 
-    def _attend_general(self, y, col0, batch, cache, page_size, out, out_col, out_scale, gate_col, gate_act):
+    def _attend_general(self, y, col0, batch, cache, page_size, out, out_col, out_scale, gate_col, gate_act, gate_group):
         """Averaged blocks and / or mixed heads.  Long portions take the sequence library's tensor-core prompt kernel when they
         fit (bf16, equal head sizes of 64 or 128, aligned rows) — with mixed heads once per value head, every head's weights on
         that head's values; every other token takes the (token, head) kernel, which reads a row's value heads side by side."""
         H, G, dv = self.heads, self.kv_heads, self.dv
         mixed = self.talk is not None
+        if mixed and gate_col is not None and gate_group != 1:
+            raise ValueError("mixed heads take a gate per entry")
         res = torch.empty(y.shape[0], H * G * dv, dtype=torch.float32, device=y.device) if mixed else out      # mixed: head g's weights on every value head
         res_col = 0 if mixed else out_col
         tok_index = None
@@ -189,7 +213,7 @@ class WindowAttention:
             all(v % 8 == 0 for v in (y.stride(0), col0, res.stride(0), res_col))
         if batch.long and fits:
             K.prompt_attention(y, col0, cache["k"], cache["v"], batch, page_size, H, G, dv, self.scale, self.window, self.keep_first, self.sink, res,
-                               res_col, pool=self.pool, pool_base=self.pool_base, every_value_head=mixed)
+                               res_col, pool=self.pool, pool_base=self.pool_base, every_value_head=mixed, chunk=self.chunk)
             if out_scale != 1.0:
                 for row0, rows, _, _ in batch.long:
                     K.scale_rows(res, row0, rows, res_col, res.shape[1] if mixed else H * dv, out_scale)
@@ -201,26 +225,26 @@ class WindowAttention:
                     n = min(per_call, G - g0)
                     K.paged_attention(y, col0, cache["k"], cache["v"], H, G, self.dk, n * dv, self.scale, self.window, self.keep_first, self.sink,
                                       batch, page_size, res, g0 * dv, out_scale, tok_index, v_row=G * dv, pool=self.pool, pool_base=self.pool_base,
-                                      v_shared=True, v_col=g0 * dv, out_head=G * dv)
+                                      v_shared=True, v_col=g0 * dv, out_head=G * dv, chunk=self.chunk)
             else:
                 K.paged_attention(y, col0, cache["k"], cache["v"], H, G, self.dk, dv, self.scale, self.window, self.keep_first, self.sink, batch,
-                                  page_size, out, out_col, out_scale, tok_index, pool=self.pool, pool_base=self.pool_base)
+                                  page_size, out, out_col, out_scale, tok_index, pool=self.pool, pool_base=self.pool_base, chunk=self.chunk)
         if mixed:
             K.mix_heads(res, self.talk, H, G, dv, out[:, out_col:], y if gate_col is not None else None, gate_col or 0, gate_act)
         elif gate_col is not None:
-            K.gate_cols(out[:, out_col:], y, gate_col, H * dv, 1, gate_act)
+            K.gate_cols(out[:, out_col:], y, gate_col, H * dv, gate_group, gate_act)
 
     def _attend_plain(self, y, col0, kc, vc, batch, cache, page_size, out, out_col, out_scale):
         tok_index = None
         aligned = all(v % 8 == 0 for v in (y.stride(0), col0, out.stride(0), out_col))
         if batch.long and y.dtype == torch.bfloat16 and self.dk == self.dv and self.dk in (64, 128) and aligned:
-            plain = self.sink is None and self.keep_first == 0 and vc is not None       # what the package's prompt kernels know
+            plain = self.sink is None and self.keep_first == 0 and self.chunk == 0 and vc is not None       # what the package's prompt kernels know
             if plain and len(batch.fresh) == len(batch.long):
                 for row0, rows in batch.fresh:
                     K.fresh_prompt_attention(y, row0, rows, col0, kc, vc, self.heads, self.kv_heads, self.dk, self.scale, self.window, out, out_col)
             else:
                 K.prompt_attention(y, col0, cache["k"], cache["v"], batch, page_size, self.heads, self.kv_heads, self.dk, self.scale, self.window,
-                                   self.keep_first, self.sink, out, out_col)
+                                   self.keep_first, self.sink, out, out_col, chunk=self.chunk)
             if out_scale != 1.0:
                 for row0, rows, _, _ in batch.long:
                     K.scale_rows(out, row0, rows, out_col, self.heads * self.dv, out_scale)
@@ -228,7 +252,7 @@ class WindowAttention:
             if tok_index.numel() == 0:
                 return
         K.paged_attention(y, col0, cache["k"], cache["v"], self.heads, self.kv_heads, self.dk, self.dv, self.scale, self.window,
-                          self.keep_first, self.sink, batch, page_size, out, out_col, out_scale, tok_index)
+                          self.keep_first, self.sink, batch, page_size, out, out_col, out_scale, tok_index, chunk=self.chunk)
 
 
 class InputConvolution:
@@ -262,7 +286,7 @@ class LatentAttentionMixer:
     """Multi-head latent attention.  Queries: c_q = rms_norm(W_dq h) w, q = W_uq c_q, per head [dn plain | dr rotated].
     Keys / values: W_dkv h = [kv_rank | dr]; c = rms_norm(first part) w is the latent, the last dr entries (rotated, not
     normed) are one key part all heads share; k_h = [W_uk,h c | shared part], v_h = W_uv,h c.  Only c and the shared part
-    are cached (one row of kv_rank + dr per token).  Rotation turns neighbouring pairs.  Scores are scaled by a given
+    are cached (one row of kv_rank + dr per token).  Rotation turns pairs of entries (`pairing`).  Scores are scaled by a given
     constant; position i sees j with 0 <= i - j < window (0: all).
 
     Computed in the absorbed form: a head's query becomes [W_uk,h^T q_plain | q_rot] (size kv_rank + dr), attention runs
@@ -278,11 +302,15 @@ class LatentAttentionMixer:
 
     q_rank 0: there is no query latent — w_down's first heads * (dn + dr) rows are the query projection itself (w_uq and
     q_norm_w are None).  dr 0 with rotation None: no rotated part, scores carry no position.  `head_gate`: w_down ends with
-    `heads` more rows, and head h's output is multiplied by that activation of row h's product (a gate per head)."""
+    `heads` more rows, and head h's output is multiplied by that activation of row h's product (a gate per head).  `entry_gate`:
+    the same with heads * dv more rows, one per entry of the concatenated heads."""
 
     def __init__(self, w_down, w_uq, w_uk, w_uv, w_o, q_norm_w, kv_norm_w, heads, dn, dr, dv, q_rank, kv_rank, scale, window, rotation, eps,
-                 page_size, shares=False, head_gate=None):
-        self.head_gate = head_gate
+                 page_size, shares=False, head_gate=None, entry_gate=None, pairing=K.PAIRS_NEIGHBOURS):
+        if head_gate is not None and entry_gate is not None:
+            raise ValueError("one output gate: per head or per entry")
+        self.gate_act, self.gate_group = (head_gate, dv) if head_gate is not None else (entry_gate, 1)
+        self.pairing = pairing
         self.w_down, self.w_uq, self.w_o, self.q_norm_w, self.kv_norm_w = w_down, w_uq, w_o, q_norm_w, kv_norm_w
         self.w_uk_rows, self.w_uv_rows = w_uk, w_uv                      # [H dn, r] / [H dv, r]: the decompressing products
         self.w_uk = w_uk.view(heads, dn, kv_rank)                       # [H][dn][r]: q_plain,h @ w_uk[h] = W_uk,h^T q_plain,h
@@ -318,8 +346,8 @@ class LatentAttentionMixer:
             out = torch.empty(T, H * self.dv, dtype=h.dtype, device=h.device)
             K.dense_prompt_attention(q2, 0, linear(c, self.w_uk_rows), linear(c, self.w_uv_rows), batch, H, H, self.dv, self.scale, self.window,
                                      None, out)
-            if self.head_gate is not None:
-                K.gate_cols(out, y, q_cols + R, H * self.dv, self.dv, self.head_gate)
+            if self.gate_act is not None:
+                K.gate_cols(out, y, q_cols + R, H * self.dv, self.gate_group, self.gate_act)
             return linear(out, self.w_o)
         cos_sin = self.rotation.table(batch) if self.rotation is not None else None
         rot_dims = self.rotation.dims if self.rotation is not None else 0
@@ -328,17 +356,18 @@ class LatentAttentionMixer:
         if self.q_rank > 0:
             cq = torch.empty(T, self.q_rank, dtype=h.dtype, device=h.device)
             K.latent_prepare(y, 0, self.q_rank, self.q_norm_w, cq, q_cols, 0 if self.shares else R, dr, rot_dims, self.kv_norm_w, cos_sin,
-                             self.eps, latent, batch.slot_of_tok)
+                             self.eps, latent, batch.slot_of_tok, pairing=self.pairing)
             q2 = linear(cq, self.w_uq)
         else:
             if not self.shares:
-                K.latent_prepare(y, 0, 0, None, None, q_cols, R, dr, rot_dims, self.kv_norm_w, cos_sin, self.eps, latent, batch.slot_of_tok)
+                K.latent_prepare(y, 0, 0, None, None, q_cols, R, dr, rot_dims, self.kv_norm_w, cos_sin, self.eps, latent, batch.slot_of_tok,
+                                 pairing=self.pairing)
             q2 = y[:, :q_cols]
         q = q2.unflatten(1, (H, dn + dr))
         qa = torch.empty(T, H, self.row, dtype=h.dtype, device=h.device)      # the absorbed queries
         torch.bmm(q[:, :, :dn].transpose(0, 1), self.w_uk, out=qa[:, :, :R].transpose(0, 1))
         if dr > 0:
-            K.rotate_pairs(q2, dn, dn + dr, qa.view(T, -1), R, self.row, H, dr, rot_dims, cos_sin)
+            K.rotate_pairs(q2, dn, dn + dr, qa.view(T, -1), R, self.row, H, dr, rot_dims, cos_sin, pairing=self.pairing)
         o = torch.empty(T, H, R, dtype=h.dtype, device=h.device)
         if h.dtype == torch.bfloat16 and K.latent_attention_fits(R, dr) and latent.stride(0) % 8 == 0:
             K.latent_prompt_attention(qa.view(T, -1), latent, H, R, dr, self.scale, self.window, batch, self.page_size, o.view(T, -1))
@@ -346,9 +375,9 @@ class LatentAttentionMixer:
             K.latent_attention(qa.view(T, -1), latent, H, R, dr, self.scale, self.window, batch, self.page_size, o.view(T, -1))
         out = torch.empty(T, H, self.dv, dtype=h.dtype, device=h.device)
         torch.bmm(o.transpose(0, 1), self.w_uv_t, out=out.transpose(0, 1))
-        if self.head_gate is not None:
+        if self.gate_act is not None:
             gate_col = q_cols + (0 if self.shares else R + dr)
-            K.gate_cols(out.view(T, H * self.dv), y, gate_col, H * self.dv, self.dv, self.head_gate)
+            K.gate_cols(out.view(T, H * self.dv), y, gate_col, H * self.dv, self.gate_group, self.gate_act)
         return linear(out.view(T, H * self.dv), self.w_o)
 
 
@@ -406,12 +435,13 @@ class GatedLinearAttentionMixer:
 
 class AttentionMixer:
     """A `WindowAttention` with its own projections: one input GEMM for q | k | v (optionally biased), attention,
-    output projection (optionally biased).  `gate_act`: w_in has heads * dv more rows after q | k | v, and the attention's
-    result is multiplied entry by entry with that activation of them before the output projection."""
+    output projection (optionally biased).  `gate_act`: w_in has heads * dv more rows after q | k | v (`gate_per_head`: one per
+    head), and the attention's result is multiplied entry by entry (head by head) with that activation of them before the
+    output projection.  Zero rows may pad w_in at its end."""
 
-    def __init__(self, attn: WindowAttention, w_in, w_out, page_size, b_in=None, b_out=None, gate_act=None):
+    def __init__(self, attn: WindowAttention, w_in, w_out, page_size, b_in=None, b_out=None, gate_act=None, gate_per_head=False):
         self.attn, self.w_in, self.w_out, self.b_in, self.b_out, self.page_size = attn, w_in, w_out, b_in, b_out, page_size
-        self.gate_act = gate_act
+        self.gate_act, self.gate_group = gate_act, attn.dv if gate_per_head else 1
 
     def alloc_cache(self, n_slots, n_token_slots, dtype, device):
         return self.attn.alloc_cache(n_slots, n_token_slots, dtype, device)
@@ -422,7 +452,8 @@ class AttentionMixer:
         if self.gate_act is None:
             self.attn.attend(y, 0, batch, cache, self.page_size, o)
         else:
-            self.attn.attend(y, 0, batch, cache, self.page_size, o, gate_col=self.attn.proj_cols, gate_act=self.gate_act)
+            self.attn.attend(y, 0, batch, cache, self.page_size, o, gate_col=self.attn.proj_cols, gate_act=self.gate_act,
+                             gate_group=self.gate_group)
         return F.linear(o, self.w_out, self.b_out)
 
 
@@ -507,7 +538,8 @@ class ParallelMixer:
 
 
 class DenseGLU:
-    """down(act(gate h) * up h) with gate and up as one GEMM."""
+    """down(act(gate h) * up h) with gate and up as one GEMM.  `act`: an activation code or a `seq_ops.GluRule` (how the two
+    halves are joined)."""
 
     def __init__(self, w_gate_up, w_down, act):
         self.w_gate_up, self.w_down, self.act = w_gate_up, w_down, act

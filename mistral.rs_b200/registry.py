@@ -54,6 +54,11 @@ def _load_kibotar(model_dir, device, dtype, **options):
     return KibotarModel.from_dir(model_dir, device, dtype, **options)
 
 
+def _load_pikasun(model_dir, device, dtype, **options):
+    from .pikasun import PikasunModel
+    return PikasunModel.from_dir(model_dir, device, dtype, **options)
+
+
 def _load_llama(model_dir, device, dtype, **options):
     """Llama-family UQFF folder (config.json + *.uqff shards + residual.safetensors) -> `model.LlamaWeights`, the object
     `model.LlamaRunner` / `model.LlamaPrefill` drive."""
@@ -72,5 +77,6 @@ register("Nisasun", _load_nisasun)
 register("Kilizen", _load_kilizen)
 register("Fosulix", _load_fosulix)
 register("Kibotar", _load_kibotar)
+register("Pikasun", _load_pikasun)
 for _name in ("LlamaForCausalLM", "MistralForCausalLM", "llama", "mistral"):
     register(_name, _load_llama)

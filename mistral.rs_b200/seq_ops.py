@@ -16,6 +16,7 @@ ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_SIGMOID, ACT_GELU_ERF, ACT_RELU_SQ = 0, 1
 GLU_CAPPED = 100
 SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
 QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_WHOLE = 0, 1, 2
+PAIRS_HALVES, PAIRS_NEIGHBOURS = 0, 1
 DTYPE_CODE = {torch.bfloat16: BF16, torch.float32: F32}
 _lib = None
 
@@ -75,7 +76,8 @@ class RmsResidualArgs(ctypes.Structure):
     _fields_ = [("src", ctypes.c_void_p), ("dst", ctypes.c_void_p), ("y", ctypes.c_void_p), ("mult", ctypes.c_float),
                 ("hist", ctypes.c_void_p), ("hist_stride", ctypes.c_int64), ("n_hist", ctypes.c_int), ("mix", ctypes.c_void_p),
                 ("mixed", ctypes.c_void_p), ("next_w", ctypes.c_void_p), ("eps", ctypes.c_float), ("next_out", ctypes.c_void_p),
-                ("dtype", ctypes.c_int), ("n_tok", ctypes.c_int), ("width", ctypes.c_int), ("post_w", ctypes.c_void_p), ("add_vec", ctypes.c_void_p)]
+                ("dtype", ctypes.c_int), ("n_tok", ctypes.c_int), ("width", ctypes.c_int), ("post_w", ctypes.c_void_p), ("add_vec", ctypes.c_void_p),
+                ("next_b", ctypes.c_void_p), ("center", ctypes.c_int), ("rows", ctypes.c_void_p)]
 
 
 class LatentPrepareArgs(ctypes.Structure):
@@ -84,7 +86,8 @@ class LatentPrepareArgs(ctypes.Structure):
                 ("kv_col", ctypes.c_int), ("kv_rank", ctypes.c_int), ("rot_dim", ctypes.c_int), ("rot_dims", ctypes.c_int),
                 ("kv_norm_w", ctypes.c_void_p), ("cos_sin", ctypes.c_void_p), ("eps", ctypes.c_float), ("cache", ctypes.c_void_p),
                 ("cache_row", ctypes.c_int64), ("slot_of_tok", ctypes.c_void_p), ("n_tok", ctypes.c_int), ("kv_out", ctypes.c_void_p),
-                ("kv_out_ld", ctypes.c_int64)]
+                ("kv_out_ld", ctypes.c_int64), ("pairing", ctypes.c_int)]
+
 
 class AttnPrepareArgs(ctypes.Structure):
     _fields_ = [("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("v", ctypes.c_void_p),
@@ -93,7 +96,8 @@ class AttnPrepareArgs(ctypes.Structure):
                 ("q_norm_w", ctypes.c_void_p), ("k_norm_w", ctypes.c_void_p), ("eps", ctypes.c_float),
                 ("heads", ctypes.c_int), ("kv_heads", ctypes.c_int), ("dk", ctypes.c_int), ("dv", ctypes.c_int),
                 ("rot_dims", ctypes.c_int), ("cos_sin", ctypes.c_void_p),
-                ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p), ("slot_of_tok", ctypes.c_void_p), ("n_tok", ctypes.c_int)]
+                ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p), ("slot_of_tok", ctypes.c_void_p), ("n_tok", ctypes.c_int),
+                ("pairing", ctypes.c_int)]
 
 
 class PagedAttentionArgs(ctypes.Structure):
@@ -104,7 +108,17 @@ class PagedAttentionArgs(ctypes.Structure):
                 ("seq_of_tok", ctypes.c_void_p), ("pos_of_tok", ctypes.c_void_p), ("tok_index", ctypes.c_void_p), ("n_tok", ctypes.c_int),
                 ("out", ctypes.c_void_p), ("out_ld", ctypes.c_int64), ("out_scale", ctypes.c_float),
                 ("k_row", ctypes.c_int64), ("v_row", ctypes.c_int64), ("pool", ctypes.c_int), ("pool_base", ctypes.c_int64),
-                ("v_shared", ctypes.c_int), ("out_f32", ctypes.c_int), ("out_head", ctypes.c_int64)]
+                ("v_shared", ctypes.c_int), ("out_f32", ctypes.c_int), ("out_head", ctypes.c_int64),
+                ("chunk", ctypes.c_int)]
+
+
+class PromptAttentionArgs(ctypes.Structure):
+    _fields_ = [("q", ctypes.c_void_p), ("q_ld", ctypes.c_int64), ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p),
+                ("out", ctypes.c_void_p), ("out_ld", ctypes.c_int64), ("portions", ctypes.c_void_p), ("n_portions", ctypes.c_int),
+                ("longest", ctypes.c_int), ("pages", ctypes.c_void_p), ("pages_ld", ctypes.c_int), ("page_size", ctypes.c_int),
+                ("heads", ctypes.c_int), ("kv_heads", ctypes.c_int), ("d", ctypes.c_int), ("scale", ctypes.c_float), ("window", ctypes.c_int),
+                ("keep_first", ctypes.c_int), ("sink", ctypes.c_void_p), ("pool", ctypes.c_int), ("pool_base", ctypes.c_int64),
+                ("every_value_head", ctypes.c_int), ("chunk", ctypes.c_int)]
 
 
 SCAN_SEGMENT = 256                  # tokens per segment when a long portion is scanned as segments side by side
@@ -391,8 +405,9 @@ def rotation_table(pos_of_tok, freq, mag):
 
 
 def attention_prepare(y, q_col, k_col, v_col, norm_mode, q_norm_w, k_norm_w, eps, heads, kv_heads, dk, dv, k_cache, v_cache, slot_of_tok,
-                      cos_sin=None, rot_dims=0):
-    """q | k | v are column ranges of y.  v_col None: the values are the keys as projected."""
+                      cos_sin=None, rot_dims=0, pairing=PAIRS_HALVES):
+    """q | k | v are column ranges of y.  v_col None: the values are the keys as projected.  pairing: which two entries of a
+    head turn together."""
     a = AttnPrepareArgs()
     ld = y.stride(0)
     a.q, a.k, a.q_ld, a.k_ld = _p(y, q_col).value, _p(y, k_col).value, ld, ld
@@ -401,25 +416,27 @@ def attention_prepare(y, q_col, k_col, v_col, norm_mode, q_norm_w, k_norm_w, eps
     a.dtype, a.norm_mode = DTYPE_CODE[y.dtype], norm_mode
     a.q_norm_w, a.k_norm_w, a.eps = _p(q_norm_w).value, _p(k_norm_w).value, eps
     a.heads, a.kv_heads, a.dk, a.dv = heads, kv_heads, dk, dv
-    a.rot_dims, a.cos_sin = rot_dims, _p(cos_sin).value
+    a.rot_dims, a.cos_sin, a.pairing = rot_dims, _p(cos_sin).value, pairing
     a.k_cache, a.v_cache, a.slot_of_tok, a.n_tok = k_cache.data_ptr(), v_cache.data_ptr(), slot_of_tok.data_ptr(), y.shape[0]
     _ok(lib().mrs_seq_attention_prepare(ctypes.byref(a), _st(y)), "attention_prepare")
 
 
 def paged_attention(y, q_col, k_cache, v_cache, heads, kv_heads, dk, dv, scale, window, keep_first, sink, batch, page_size, out, out_col=0,
-                    out_scale=1.0, tok_index=None, k_row=0, v_row=0, pool=0, pool_base=0, v_shared=False, v_col=0, out_head=0):
+                    out_scale=1.0, tok_index=None, k_row=0, v_row=0, pool=0, pool_base=0, v_shared=False, v_col=0, out_head=0,
+                    chunk=0):
     """Every token of the step (or those listed in tok_index) against the pages of its sequence: position i sees j <= i
     with i - j < window (0: all) or j < keep_first; sink [heads] f32 or None.  k_row / v_row: elements between the cache
     rows of neighbouring slots (0: kv_heads * dk / kv_heads * dv).  pool > 0: besides the window, one averaged entry per
     block of `pool` positions wholly before it, read from cache rows pool_base.. (`pool_blocks`).  v_shared: every head
     reads value columns [v_col, v_col + dv) of a row — dv is then several (or all) value heads side by side, and out_head the
-    distance between the heads of an output row.  An f32 `out` is written as f32 whatever the activation type."""
+    distance between the heads of an output row.  An f32 `out` is written as f32 whatever the activation type.
+    chunk > 0: a position sees only its own chunk of `chunk` positions, counted from position 0."""
     a = PagedAttentionArgs()
     a.k_row, a.v_row = int(k_row), int(v_row)
     a.pool, a.pool_base, a.v_shared = int(pool), int(pool_base), int(bool(v_shared))
     a.out_f32 = int(out.dtype == torch.float32 and y.dtype != torch.float32)
     a.q, a.q_ld, a.k_cache, a.v_cache = _p(y, q_col).value, y.stride(0), k_cache.data_ptr(), _p(v_cache, int(v_col)).value
-    a.out_head = int(out_head)
+    a.out_head, a.chunk = int(out_head), int(chunk)
     a.dtype, a.heads, a.kv_heads, a.dk, a.dv = DTYPE_CODE[y.dtype], heads, kv_heads, dk, dv
     a.scale, a.window, a.keep_first, a.sink = scale, int(window), int(keep_first), _p(sink).value
     a.pages, a.pages_ld, a.page_size = batch.pages.data_ptr(), batch.pages.shape[1], page_size
@@ -474,15 +491,20 @@ def gate_cols(x, gate, gate_col, cols, group, act):
 
 
 def prompt_attention(y, q_col, k_cache, v_cache, batch, page_size, heads, kv_heads, d, scale, window, keep_first, sink, out, out_col=0, pool=0,
-                     pool_base=0, every_value_head=False):
+                     pool_base=0, every_value_head=False, chunk=0):
     """The long portions of the step (batch.long: fresh or continued) on tensor cores: queries from their rows of y, keys
     and values from the pages (bf16, head size 64 or 128).  pool / pool_base: averaged blocks before the window, as for
-    `paged_attention`.  every_value_head: `out` is f32 [T, heads * kv_heads * d], every head's weights on every value head."""
-    _ok(lib().mrs_seq_prompt_attention_pooled(_p(y, q_col), _l(y.stride(0)), _p(k_cache), _p(v_cache), _p(out, out_col), _l(out.stride(0)),
-                                              _p(batch.long_rows), _i(len(batch.long)), _i(max(n for _, n, _, _ in batch.long)), _p(batch.pages),
-                                              _i(batch.pages.shape[1]), _i(page_size), _i(heads), _i(kv_heads), _i(d), _f(scale), _i(int(window)),
-                                              _i(int(keep_first)), _p(sink), _i(int(pool)), _l(int(pool_base)), _i(int(bool(every_value_head))),
-                                              _st(y)), "prompt_attention")
+    `paged_attention`.  every_value_head: `out` is f32 [T, heads * kv_heads * d], every head's weights on every value head.
+    chunk > 0: a position sees only its own chunk of `chunk` positions, counted from position 0."""
+    a = PromptAttentionArgs()
+    a.q, a.q_ld, a.k_cache, a.v_cache = _p(y, q_col).value, y.stride(0), k_cache.data_ptr(), v_cache.data_ptr()
+    a.out, a.out_ld = _p(out, out_col).value, out.stride(0)
+    a.portions, a.n_portions, a.longest = batch.long_rows.data_ptr(), len(batch.long), max(n for _, n, _, _ in batch.long)
+    a.pages, a.pages_ld, a.page_size = batch.pages.data_ptr(), batch.pages.shape[1], page_size
+    a.heads, a.kv_heads, a.d, a.scale = heads, kv_heads, d, float(scale)
+    a.window, a.keep_first, a.sink = int(window), int(keep_first), _p(sink).value
+    a.pool, a.pool_base, a.every_value_head, a.chunk = int(pool), int(pool_base), int(bool(every_value_head)), int(chunk)
+    _ok(lib().mrs_seq_prompt_attention_general(ctypes.byref(a), _st(y)), "prompt_attention")
 
 
 # ---- stabilised matrix memory ---------------------------------------------------------------------------
@@ -553,11 +575,13 @@ def embed_pair(table, pairs, ids, scale, buckets, mul_prev, mul_cur, prev_state,
 
 
 def rms_residual(src, y=None, mult=1.0, dst=None, hist=None, n_hist=0, mix=None, mixed=None, next_w=None, eps=0.0, dtype=None, post_w=None,
-                 add_vec=None):
+                 add_vec=None, next_b=None, center=False, rows=None):
     """One pass over an f32 residual [T, W]: v = src + mult * y (y first RMS-normed with post_w when given) + add_vec [W] -> dst;
     v = sum_j mix[j] * hist[j] (hist f32 [>= n_hist, T, W], dst may be one of its entries) -> mixed; returns rms_norm(v) * next_w
-    in the activation type when next_w is given."""
+    in the activation type when next_w is given — with `center` a layer norm (mean taken off) and with next_b a bias.  rows: the
+    norm of these rows of src only (nothing else then happens)."""
     T, W = src.shape
+    T = T if rows is None else rows.numel()
     dtype = y.dtype if y is not None else dtype
     out = torch.empty(T, W, dtype=dtype, device=src.device) if next_w is not None else None
     a = RmsResidualArgs()
@@ -567,14 +591,23 @@ def rms_residual(src, y=None, mult=1.0, dst=None, hist=None, n_hist=0, mix=None,
     a.mixed, a.next_w, a.eps, a.next_out = _p(mixed).value, _p(next_w).value, float(eps), _p(out).value
     a.dtype, a.n_tok, a.width = DTYPE_CODE[dtype], T, W
     a.post_w, a.add_vec = _p(post_w).value, _p(add_vec).value
+    a.next_b, a.center, a.rows = _p(next_b).value, int(bool(center)), _p(rows).value
     _ok(lib().mrs_seq_rms_residual(ctypes.byref(a), _st(src)), "rms_residual")
     return out
 
 
+def soft_cap(x, scale, cap):
+    """f32 cap * tanh(scale * x / cap) (cap 0: scale * x): logits with a multiplier and a soft cap."""
+    out = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+    _ok(lib().mrs_seq_soft_cap(_p(x), _i(DTYPE_CODE[x.dtype]), _f(scale), _f(cap), _l(x.numel()), _p(out), _st(x)), "soft_cap")
+    return out
+
+
 # ---- attention through a shared latent -----------------------------------------------------------------------
-def latent_prepare(y, q_col, q_rank, q_norm_w, q_out, kv_col, kv_rank, rot_dim, rot_dims, kv_norm_w, cos_sin, eps, cache, slot_of_tok, kv_out=None):
+def latent_prepare(y, q_col, q_rank, q_norm_w, q_out, kv_col, kv_rank, rot_dim, rot_dims, kv_norm_w, cos_sin, eps, cache, slot_of_tok, kv_out=None,
+                   pairing=PAIRS_NEIGHBOURS):
     """From the columns of y: q_out = rms_norm(query latent) * w; cache[slot] = rms_norm(key/value latent) * w | the shared key
-    part turned in neighbouring pairs.  kv_rank 0: only the query part.  kv_out [T, >= kv_rank]: the normed latent also as dense rows."""
+    part turned in pairs (`pairing`).  kv_rank 0: only the query part.  kv_out [T, >= kv_rank]: the normed latent also as dense rows."""
     a = LatentPrepareArgs()
     a.y, a.y_ld, a.dtype = _p(y).value, y.stride(0), DTYPE_CODE[y.dtype]
     a.q_col, a.q_rank, a.q_norm_w = int(q_col), int(q_rank), _p(q_norm_w).value
@@ -584,17 +617,18 @@ def latent_prepare(y, q_col, q_rank, q_norm_w, q_out, kv_col, kv_rank, rot_dim, 
     a.kv_norm_w, a.cos_sin, a.eps = _p(kv_norm_w).value, _p(cos_sin).value, float(eps)
     if kv_rank:
         a.cache, a.cache_row, a.slot_of_tok = _p(cache).value, cache.stride(0), _p(slot_of_tok).value
-    a.n_tok = y.shape[0]
+    a.n_tok, a.pairing = y.shape[0], pairing
     if kv_out is not None:
         a.kv_out, a.kv_out_ld = _p(kv_out).value, kv_out.stride(0)
     _ok(lib().mrs_seq_latent_prepare(ctypes.byref(a), _st(y)), "latent_prepare")
 
 
-def rotate_pairs(src, src_col, src_head, dst, dst_col, dst_head, heads, dims, rot_dims, cos_sin):
+def rotate_pairs(src, src_col, src_head, dst, dst_col, dst_head, heads, dims, rot_dims, cos_sin, pairing=PAIRS_NEIGHBOURS):
     """dst[t, dst_col + h * dst_head + d] = src[t, src_col + h * src_head + d], d < dims, the first rot_dims turned in
-    neighbouring pairs by cos_sin [T, rot_dims / 2, 2]."""
-    _ok(lib().mrs_seq_rotate_pairs(_p(src, src_col), _l(src.stride(0)), _l(src_head), _p(dst, dst_col), _l(dst.stride(0)), _l(dst_head),
-                                   _i(DTYPE_CODE[src.dtype]), _i(heads), _i(dims), _i(rot_dims), _p(cos_sin), _i(src.shape[0]), _st(src)),
+    pairs (`pairing`) by cos_sin [T, rot_dims / 2, 2]."""
+    _ok(lib().mrs_seq_rotate_heads(_p(src, src_col), _l(src.stride(0)), _l(src_head), _p(dst, dst_col), _l(dst.stride(0)), _l(dst_head),
+                                   _i(DTYPE_CODE[src.dtype]), _i(heads), _i(dims), _i(rot_dims), _i(pairing), _p(cos_sin), _i(src.shape[0]),
+                                   _st(src)),
         "rotate_pairs")
 
 
