@@ -265,6 +265,10 @@ typedef struct {
   int out_f32;            /* != 0: out is f32 whatever the activation type */
   int64_t out_head;       /* elements between the heads of an output row; 0: dv.  With v_shared, a call may cover a column range of
                              the value heads (v_cache advanced to it) and write the same range of every head's output */
+  const void *gate;       /* NULL: none; else the result is multiplied by gate_act(gate[t][(h * dv + c) / gate_group]), gate of the
+                             activation type with row stride gate_ld, gate_group 1 or dv (not with v_shared) */
+  int64_t gate_ld;
+  int gate_group, gate_act;
   int chunk;              /* > 0: position i sees j only in its own chunk, floor(i / chunk) == floor(j / chunk), chunks counted from
                              position 0 of the sequence (combines with window; keep_first and pool must be 0) */
 } mrs_seq_paged_attention_args;
@@ -316,8 +320,40 @@ typedef struct {
   int pool;
   int64_t pool_base;
   int every_value_head, chunk;
+  const void *gate;       /* as in mrs_seq_paged_attention_args (not with every_value_head) */
+  int64_t gate_ld;
+  int gate_group, gate_act;
 } mrs_seq_prompt_attention_args;
 int mrs_seq_prompt_attention_general(const mrs_seq_prompt_attention_args *args, int64_t stream);
+/* Causal attention of segments on the 5th-gen tensor cores over DENSE keys and values (bf16): segments [n][4] = first query
+ * row (of q / out / gate), query rows, first key row (of k / k_shared / v), keys that lie before the first query (they are the
+ * first of the segment's key rows); query r of a segment sees its first past + r + 1 keys.  q [q_rows, heads, dn + dr], k [k_rows,
+ * kv_heads, dn], v [k_rows, kv_heads, dv]; dr > 0: one further key part k_shared [k_rows, dr] that all heads share, scored by the
+ * queries' last dr entries.  gate (NULL: none): the result is multiplied by gate_act(gate[row][(h * dv + d) / gate_group]),
+ * gate_group 1 or dv.  scale > 0.  *_ld: elements between rows (multiples of 8; pointers 16-byte aligned).  Every key row in
+ * [first key row, first key row + past + query rows) and the rows of the same tile behind it must hold finite values. */
+typedef struct {
+  const void *q, *k, *k_shared, *v;
+  int64_t q_ld, k_ld, k_shared_ld, v_ld;
+  int64_t q_rows, k_rows;
+  void *out;
+  int64_t out_ld;
+  const int32_t *segments;
+  int n_segments, longest;
+  int heads, kv_heads, dn, dr, dv;
+  float scale;
+  const void *gate;
+  int64_t gate_ld;
+  int gate_group, gate_act;
+} mrs_seq_prompt_attention_tc_args;
+int mrs_seq_prompt_attention_tc(const mrs_seq_prompt_attention_tc_args *args, int64_t stream);
+/* head sizes the call above takes: dn a multiple of 16 up to 128, dr a multiple of 8 up to 64, dv a multiple of 8 up to 128 */
+int mrs_seq_prompt_attention_tc_fits(int dn, int dr, int dv);
+/* non-zero when a wait inside the kernel ever ran out (synchronises; negative: a CUDA error) */
+int mrs_seq_prompt_attention_tc_timeouts(void);
+/* Cached rows of sequences -> dense rows: runs [n][4] = row of `pages`, first position, positions, first row of out. */
+int mrs_seq_gather_rows(const void *cache, int64_t cache_row_bytes, int row_bytes, const int32_t *runs, int n_runs, int longest,
+                        const int32_t *pages, int pages_ld, int page_size, void *out, int64_t out_row_bytes, int64_t stream);
 /* ---- attention through a shared latent ----------------------------------------------------------------- */
 /* Per token, from the columns of one projection y (row stride y_ld, activation type), any part optional:
  *   q_out[t] = rms_norm(y[t][q_col : q_col + q_rank]) * q_norm_w                      (the query latent, activation type)
@@ -325,8 +361,10 @@ int mrs_seq_prompt_attention_general(const mrs_seq_prompt_attention_args *args, 
  *   cache[slot(t)][kv_rank : kv_rank + rot_dim] = turn(y[t][kv_col + kv_rank : ...])     (the key part all heads share)
  * turn: pair i < rot_dims / 2 (`pairing`) rotates by cos_sin[t][i] (f32 [n_tok, rot_dims / 2, 2]); the rest pass.
  * cache rows are cache_row elements apart.  q_rank 0: no query part; kv_rank 0: no cache part.  kv_out (optional): the normed
- * key/value latent also goes to kv_out[t][0 : kv_rank] (row stride kv_out_ld), for callers that decompress keys and values
- * of the step's own tokens with a matrix product. */
+ * key/value latent also goes to kv_out[t][0 : kv_rank] (row stride kv_out_ld; with room for it the turned key part follows), for callers that decompress keys and values
+ * of the step's own tokens with a matrix product.  rq_heads > 0 (optional): the queries' rotated parts turn in the same pass,
+ * rq_out[t][h * rq_out_head + d] = turn(y[t][rq_col + h * rq_head + d]) for d < rot_dim, h < rq_heads (rq_out row stride
+ * rq_out_ld; writing back into y is fine). */
 typedef struct {
   const void *y;
   int64_t y_ld;
@@ -346,6 +384,10 @@ typedef struct {
   void *kv_out;
   int64_t kv_out_ld;
   int pairing;
+  int rq_heads, rq_col;
+  int64_t rq_head;
+  void *rq_out;
+  int64_t rq_out_ld, rq_out_head;
 } mrs_seq_latent_prepare_args;
 int mrs_seq_latent_prepare(const mrs_seq_latent_prepare_args *args, int64_t stream);
 /* out[t][h][0:dims] = in[t][h][0:dims] with entries (2i, 2i + 1), i < rot_dims / 2, rotated by cos_sin[t][i], the rest
@@ -368,6 +410,26 @@ int mrs_seq_latent_attention(const void *q, int64_t q_ld, const void *cache, int
                              const int32_t *portions, const int32_t *cu_tok, const int32_t *past, int n_portions, int longest,
                              const int32_t *pages, int pages_ld, int page_size, int heads, int kv_rank, int rot_dim, float scale,
                              int window, int64_t stream);
+/* The same in one structure, with the key tiles of a row tile shared by `splits` CTAs (<= 1: not) when row tiles alone do not
+ * fill the GPU.  scratch: f32, as many floats as the plan asks for, 16-byte aligned.  The plan returns the split count for a
+ * step whose sequences reach at most max_keys positions (constant for a captured step). */
+typedef struct {
+  const void *q;
+  int64_t q_ld;
+  const void *cache;
+  int64_t cache_row;
+  void *out;
+  int64_t out_ld;
+  const int32_t *portions, *cu_tok, *past;
+  int n_portions, longest;
+  const int32_t *pages;
+  int pages_ld, page_size, heads, kv_rank, rot_dim;
+  float scale;
+  int window, splits;
+  float *scratch;
+} mrs_seq_latent_attention_args;
+int mrs_seq_latent_attention_general(const mrs_seq_latent_attention_args *args, int64_t stream);
+int mrs_seq_latent_attention_plan(int n_portions, int longest, int heads, int kv_rank, int max_keys, int64_t *scratch_floats);
 
 /* x[r][c] *= scale for r < rows, c < cols (row stride ld) */
 int mrs_seq_scale_rows(void *x, int64_t ld, int dtype, int rows, int cols, float scale, int64_t stream);

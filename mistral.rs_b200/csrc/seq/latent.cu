@@ -28,6 +28,26 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const mrs_seq_laten
     T *dst = (T *)a.q_out + (int64_t)t * a.q_out_ld;
     for (int c = threadIdx.x; c < a.q_rank; c += blockDim.x) dst[c] = from_f32<T>(to_f32<T>(src[c]) * inv * a.q_norm_w[c]);
   }
+  if (a.rq_heads > 0) {           // the queries' rotated parts
+    const int half = a.cos_sin ? a.rot_dims / 2 : 0;
+    const float2 *cs = (const float2 *)a.cos_sin + (int64_t)t * half;
+    T *out = (T *)a.rq_out + (int64_t)t * a.rq_out_ld;
+    const int rest = a.rot_dim - 2 * half, items = half + rest;       // a pair, or an entry that passes
+    for (int e = threadIdx.x; e < a.rq_heads * items; e += blockDim.x) {
+      const int h = e / items, i = e % items;
+      const T *s = y + a.rq_col + (int64_t)h * a.rq_head;
+      T *d = out + (int64_t)h * a.rq_out_head;
+      if (i < half) {
+        const int iu = pair_u(i, a.pairing), iv = pair_v(i, half, a.pairing);
+        const float u = to_f32<T>(s[iu]), v = to_f32<T>(s[iv]);
+        const float2 c = cs[i];
+        d[iu] = from_f32<T>(u * c.x - v * c.y);
+        d[iv] = from_f32<T>(v * c.x + u * c.y);
+      } else {
+        d[half + i] = s[half + i];
+      }
+    }
+  }
   if (a.kv_rank <= 0) return;
   const int64_t slot = a.slot_of_tok[t];
   if (slot < 0) return;       // uniform over the block
@@ -49,14 +69,22 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const mrs_seq_laten
   const float2 *cs = (const float2 *)a.cos_sin + (int64_t)t * half;
   src += a.kv_rank;
   dst += a.kv_rank;
+  dense = dense && a.kv_out_ld >= a.kv_rank + a.rot_dim ? dense + a.kv_rank : nullptr;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     const int iu = pair_u(i, a.pairing), iv = pair_v(i, half, a.pairing);
     const float u = to_f32<T>(src[iu]), v = to_f32<T>(src[iv]);
     const float2 c = cs[i];
     dst[iu] = from_f32<T>(u * c.x - v * c.y);
     dst[iv] = from_f32<T>(v * c.x + u * c.y);
+    if (dense) {
+      dense[iu] = dst[iu];
+      dense[iv] = dst[iv];
+    }
   }
-  for (int d = 2 * half + threadIdx.x; d < a.rot_dim; d += blockDim.x) dst[d] = src[d];
+  for (int d = 2 * half + threadIdx.x; d < a.rot_dim; d += blockDim.x) {
+    dst[d] = src[d];
+    if (dense) dense[d] = src[d];
+  }
 }
 
 // one CTA per token, all heads: out[t][h][:dims] = in[t][h][:dims] with the first rot_dims entries turned in pairs.  In place
@@ -94,11 +122,13 @@ using namespace seq;
 extern "C" int mrs_seq_latent_prepare(const mrs_seq_latent_prepare_args *args, int64_t stream) {
   const mrs_seq_latent_prepare_args &a = *args;
   if (a.n_tok <= 0) return 0;
-  if (!a.y || a.q_rank < 0 || a.kv_rank < 0 || (a.q_rank == 0 && a.kv_rank == 0)) return -2;
+  if (!a.y || a.q_rank < 0 || a.kv_rank < 0 || (a.q_rank == 0 && a.kv_rank == 0 && a.rq_heads <= 0)) return -2;
+  if (a.rq_heads > 0 && (!a.rq_out || a.rot_dim <= 0)) return -2;
   if (a.q_rank > 0 && (!a.q_norm_w || !a.q_out)) return -2;
   if (a.kv_rank > 0 && (!a.kv_norm_w || !a.cache || !a.slot_of_tok || a.rot_dim < 0 || a.cache_row < a.kv_rank + a.rot_dim)) return -2;
-  if (a.kv_rank > 0 && a.cos_sin && (a.rot_dims < 2 || a.rot_dims % 2 || a.rot_dims > a.rot_dim)) return -2;
-  const int widest = a.q_rank > a.kv_rank ? a.q_rank : a.kv_rank;
+  if ((a.kv_rank > 0 || a.rq_heads > 0) && a.cos_sin && (a.rot_dims < 2 || a.rot_dims % 2 || a.rot_dims > a.rot_dim)) return -2;
+  int widest = a.q_rank > a.kv_rank ? a.q_rank : a.kv_rank;
+  if (a.rq_heads > 0 && a.rq_heads * a.rot_dim / 2 > widest) widest = a.rq_heads * a.rot_dim / 2;
   const int th = widest >= 1024 ? 256 : (widest >= 256 ? 128 : 64);
   SEQ_DISPATCH_DTYPE(a.dtype, (latent_prepare_kernel<T><<<a.n_tok, th, 0, (cudaStream_t)stream>>>(a)));
   return launch_status();

@@ -13,6 +13,8 @@
 //   C  O = O * rescale + P V: warp w takes row tile w % MT and one of 8 / MT column groups of the kv_rank output columns
 //      (at most 128 columns, 64 accumulator registers), V fragments are transposed loads of the same key tile.
 // MT = 4, 2, 1 for kv_rank up to 256, 512, 1024.  bf16 only; dk and kv_rank multiples of 8.
+// When the row tiles alone do not fill the GPU (decoding), `splits` CTAs share a row tile's key tiles and leave their maxima,
+// sums and unscaled outputs as f32 partial results, which a second kernel merges.
 // A decoded token is a portion of one token: its heads are the rows of one tile and the window's latents are fetched once
 // for all of them, where a (token, head) kernel fetches them once per head.
 #include "../mma_common.cuh"
@@ -22,7 +24,7 @@
 namespace seql {
 using namespace mrs;
 
-constexpr int BN = 64, WARPS = 8, THREADS = WARPS * 32, SS = BN + 4, PB = BN * 2 + 16, MAX_TILES = 16;
+constexpr int BN = 64, WARPS = 8, THREADS = WARPS * 32, SS = BN + 4, PB = BN * 2 + 16, MAX_TILES = 16, MAX_SPLITS = 32;
 
 struct Params {
   const __nv_bfloat16 *q, *cache;
@@ -35,6 +37,8 @@ struct Params {
   int H, DK, R;
   float scale_log2;
   int window;                  // <= 0: every earlier position
+  int splits;                  // CTAs side by side over the key tiles of a row tile; > 1: partial results, merged afterwards
+  float *part_o, *part_ml;     // [n][splits][rows of the grid][R] unscaled sums, and [..][2] (running maximum, sum)
 };
 
 template <int MT>
@@ -57,7 +61,13 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(const 
   if (row0 >= n_rows) return;
   const int tok_lo = row0 / p.H, tok_hi = min(len - 1, (row0 + BM - 1) / p.H);
   const int k_first = p.window > 0 ? max(0, past + tok_lo - p.window + 1) : 0, k_end = past + tok_hi + 1;
-  const int nt = (k_end - k_first + BN - 1) / BN;
+  const int nt_all = (k_end - k_first + BN - 1) / BN, per_split = (nt_all + p.splits - 1) / p.splits;
+  const int t_begin = blockIdx.z * per_split, nt = min(nt_all, t_begin + per_split);
+  const int64_t part_row0 = ((int64_t)(b * p.splits + blockIdx.z) * gridDim.x + blockIdx.x) * BM;
+  if (t_begin >= nt) {                   // fewer key tiles than splits: an empty share
+    for (int r = threadIdx.x; r < BM; r += THREADS) *(float2 *)(p.part_ml + (part_row0 + r) * 2) = make_float2(-INFINITY, 0.f);
+    return;
+  }
 
   auto load_tile = [&](int t, int buf) {
     const int t0 = k_first + t * BN;
@@ -78,7 +88,7 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(const 
     cp_async16(sq + row * kstride + ch * 16, p.q + (int64_t)(tok0 + gg / p.H) * p.q_ld + (int64_t)(gg % p.H) * p.DK + ch * 8, ok);
   }
   cp_async_commit();
-  load_tile(0, 0);
+  load_tile(t_begin, 0);
 
   // phase A / C roles
   const int mt = warp % MT, grp = warp / MT;
@@ -94,8 +104,8 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(const 
   const int bpos = past + min(bg, n_rows - 1) / p.H;
   float m_run = -INFINITY, l_run = 0.f;
 
-  for (int t = 0; t < nt; t++) {
-    const int buf = t & 1;
+  for (int t = t_begin; t < nt; t++) {
+    const int buf = (t - t_begin) & 1;
     cp_async_wait<0>();
     __syncthreads();                       // tile t (and Q) landed; everyone is done with tile t - 1
     if (t + 1 < nt) load_tile(t + 1, buf ^ 1);
@@ -181,8 +191,23 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(const 
       }
     }
   }
-  if (bsub == 0) sl[brow] = l_run;
+  if (bsub == 0) {
+    sl[brow] = l_run;
+    if (p.splits > 1) *(float2 *)(p.part_ml + (part_row0 + brow) * 2) = make_float2(m_run, l_run);
+  }
   __syncthreads();
+  if (p.splits > 1) {
+    float *o0 = p.part_o + (part_row0 + mt * 16 + (lane >> 2)) * p.R, *o1 = o0 + (int64_t)8 * p.R;
+#pragma unroll
+    for (int i = 0; i < MAX_TILES; i++) {
+      if (i < my_tiles) {
+        const int col = (tile0 + i) * 8 + 2 * (lane & 3);
+        *(float2 *)(o0 + col) = make_float2(oacc[i][0], oacc[i][1]);
+        *(float2 *)(o1 + col) = make_float2(oacc[i][2], oacc[i][3]);
+      }
+    }
+    return;
+  }
   const int ra = mt * 16 + (lane >> 2);
   const float l0 = sl[ra], l1 = sl[ra + 8];
   const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
@@ -197,6 +222,51 @@ __global__ void __launch_bounds__(THREADS, 1) latent_attention_mma_kernel(const 
       if (o1) *(uint32_t *)(o1 + col) = pack2<T>(oacc[i][2] * inv1, oacc[i][3] * inv1);
     }
   }
+}
+
+// One CTA per (token, head) row: the splits' partial sums weighted by 2^(their maximum - the row's) and divided by the row's sum.
+__global__ void __launch_bounds__(128) latent_merge_kernel(const Params p, int rows_cap) {
+  const int b = blockIdx.y, g = blockIdx.x;
+  const int tok0 = p.portions ? p.portions[4 * b] : p.cu_tok[b], len = p.portions ? p.portions[4 * b + 1] : p.cu_tok[b + 1] - tok0;
+  if (g >= len * p.H) return;
+  __shared__ float w[MAX_SPLITS];
+  const float *ml = p.part_ml + ((int64_t)b * p.splits * rows_cap + g) * 2;
+  if (threadIdx.x < 32) {
+    const bool mine = (int)threadIdx.x < p.splits;
+    const float2 v = mine ? *(const float2 *)(ml + (int64_t)threadIdx.x * rows_cap * 2) : make_float2(-INFINITY, 0.f);
+    float mx = v.x;
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, m));
+    const float e = v.x == -INFINITY ? 0.f : exp2f(v.x - mx);
+    float l = e * v.y;
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) l += __shfl_xor_sync(0xffffffffu, l, m);
+    w[threadIdx.x] = e / l;
+  }
+  __syncthreads();
+  const float *src = p.part_o + ((int64_t)b * p.splits * rows_cap + g) * p.R;
+  __nv_bfloat16 *dst = p.o + (int64_t)(tok0 + g / p.H) * p.o_ld + (int64_t)(g % p.H) * p.R;
+  for (int c = threadIdx.x * 4; c < p.R; c += 512) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < p.splits; s++) {
+      const float ws = w[s];
+      if (ws == 0.f) continue;           // an empty share holds no sums
+      const float4 v = *(const float4 *)(src + (int64_t)s * rows_cap * p.R + c);
+      acc.x = fmaf(ws, v.x, acc.x); acc.y = fmaf(ws, v.y, acc.y); acc.z = fmaf(ws, v.z, acc.z); acc.w = fmaf(ws, v.w, acc.w);
+    }
+    uint2 pk;
+    pk.x = pack2<__nv_bfloat16>(acc.x, acc.y);
+    pk.y = pack2<__nv_bfloat16>(acc.z, acc.w);
+    *(uint2 *)(dst + c) = pk;
+  }
+}
+
+// row tiles per CTA: as many as the output columns allow, but no more than the longest portion fills (a decoded token's heads
+// are one or two tiles: all eight warps then split its keys and columns)
+static int row_tiles(int longest, int heads, int kv_rank) {
+  const int64_t rows = (int64_t)longest * heads;
+  const int by_rank = kv_rank <= 256 ? 4 : (kv_rank <= 512 ? 2 : 1), by_rows = rows <= 16 ? 1 : (rows <= 32 ? 2 : 4);
+  return by_rank < by_rows ? by_rank : by_rows;
 }
 
 static size_t smem_bytes(int mt, int dk) {
@@ -214,7 +284,9 @@ static int launch(const Params &p, int n, int longest, cudaStream_t st) {
     if (e != cudaSuccess) return (int)e;
     allowed = bytes;
   }
-  kern<<<dim3((longest * p.H + 16 * MT - 1) / (16 * MT), n), THREADS, bytes, st>>>(p);
+  const int tiles = (int)(((int64_t)longest * p.H + 16 * MT - 1) / (16 * MT));
+  kern<<<dim3(tiles, n, p.splits), THREADS, bytes, st>>>(p);
+  if (p.splits > 1) latent_merge_kernel<<<dim3(longest * p.H, n), 128, 0, st>>>(p, tiles * 16 * MT);
   return (int)cudaGetLastError();
 }
 
@@ -227,27 +299,56 @@ extern "C" int mrs_seq_latent_attention_fits(int kv_rank, int rot_dim) {
   return seql::smem_bytes(mt, dk) <= 220 * 1024 ? 1 : 0;
 }
 
+extern "C" int mrs_seq_latent_attention_plan(int n_portions, int longest, int heads, int kv_rank, int max_keys, int64_t *scratch_floats) {
+  *scratch_floats = 0;
+  if (n_portions <= 0 || longest <= 0 || heads <= 0 || kv_rank <= 0) return 1;
+  const int bm = 16 * seql::row_tiles(longest, heads, kv_rank);
+  const int64_t tiles = ((int64_t)longest * heads + bm - 1) / bm, ctas = tiles * n_portions;
+  int64_t splits = 148 / ctas;
+  const int64_t by_keys = (max_keys + 2 * seql::BN - 1) / (2 * seql::BN);       // two key tiles per share at the longest reach
+  if (splits > by_keys) splits = by_keys;
+  if (splits > seql::MAX_SPLITS) splits = seql::MAX_SPLITS;
+  if (splits < 2) return 1;
+  *scratch_floats = n_portions * splits * tiles * bm * (kv_rank + 2);
+  return (int)splits;
+}
+
+extern "C" int mrs_seq_latent_attention_general(const mrs_seq_latent_attention_args *args, int64_t stream) {
+  const mrs_seq_latent_attention_args &a = *args;
+  if (a.n_portions <= 0 || a.longest <= 0) return 0;
+  if (a.heads <= 0 || (!a.portions && (!a.cu_tok || !a.past)) || !a.pages || a.page_size <= 0 ||
+      !mrs_seq_latent_attention_fits(a.kv_rank, a.rot_dim))
+    return -2;
+  if ((a.q_ld | a.out_ld | a.cache_row) % 8 || (((uintptr_t)a.q | (uintptr_t)a.cache | (uintptr_t)a.out) & 15)) return -3;
+  if (a.splits > 1 && (!a.scratch || a.splits > seql::MAX_SPLITS || ((uintptr_t)a.scratch & 15))) return -2;
+  seql::Params p = {};
+  p.q = (const __nv_bfloat16 *)a.q; p.cache = (const __nv_bfloat16 *)a.cache; p.o = (__nv_bfloat16 *)a.out;
+  p.q_ld = a.q_ld; p.o_ld = a.out_ld; p.cache_row = a.cache_row;
+  p.portions = a.portions; p.cu_tok = a.cu_tok; p.past = a.past; p.pages = a.pages; p.pages_ld = a.pages_ld; p.page_size = a.page_size;
+  p.H = a.heads; p.DK = a.kv_rank + a.rot_dim; p.R = a.kv_rank;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.window = a.window;
+  const int mt = seql::row_tiles(a.longest, a.heads, a.kv_rank);
+  p.splits = a.splits > 1 ? a.splits : 1;
+  if (p.splits > 1) {
+    const int64_t tiles = ((int64_t)a.longest * a.heads + 16 * mt - 1) / (16 * mt);
+    p.part_o = a.scratch;
+    p.part_ml = a.scratch + (int64_t)a.n_portions * p.splits * tiles * 16 * mt * a.kv_rank;
+  }
+  cudaStream_t st = (cudaStream_t)stream;
+  if (mt == 4) return seql::launch<4>(p, a.n_portions, a.longest, st);
+  if (mt == 2) return seql::launch<2>(p, a.n_portions, a.longest, st);
+  return seql::launch<1>(p, a.n_portions, a.longest, st);
+}
+
 extern "C" int mrs_seq_latent_attention(const void *q, int64_t q_ld, const void *cache, int64_t cache_row, void *out, int64_t out_ld,
                                         const int32_t *portions, const int32_t *cu_tok, const int32_t *past, int n_portions, int longest,
                                         const int32_t *pages, int pages_ld, int page_size, int heads, int kv_rank, int rot_dim, float scale,
                                         int window, int64_t stream) {
-  if (n_portions <= 0 || longest <= 0) return 0;
-  if (heads <= 0 || (!portions && (!cu_tok || !past)) || !pages || page_size <= 0 || !mrs_seq_latent_attention_fits(kv_rank, rot_dim)) return -2;
-  if ((q_ld | out_ld | cache_row) % 8 || (((uintptr_t)q | (uintptr_t)cache | (uintptr_t)out) & 15)) return -3;
-  seql::Params p = {};
-  p.q = (const __nv_bfloat16 *)q; p.cache = (const __nv_bfloat16 *)cache; p.o = (__nv_bfloat16 *)out;
-  p.q_ld = q_ld; p.o_ld = out_ld; p.cache_row = cache_row;
-  p.portions = portions; p.cu_tok = cu_tok; p.past = past; p.pages = pages; p.pages_ld = pages_ld; p.page_size = page_size;
-  p.H = heads; p.DK = kv_rank + rot_dim; p.R = kv_rank;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window;
-  cudaStream_t st = (cudaStream_t)stream;
-  // row tiles per CTA: as many as the output columns allow, but no more than the longest portion fills (a decoded token's
-  // heads are one or two tiles: all eight warps then split its keys and columns)
-  const int64_t rows = (int64_t)longest * heads;
-  const int by_rank = kv_rank <= 256 ? 4 : (kv_rank <= 512 ? 2 : 1), by_rows = rows <= 16 ? 1 : (rows <= 32 ? 2 : 4);
-  const int mt = by_rank < by_rows ? by_rank : by_rows;
-  if (mt == 4) return seql::launch<4>(p, n_portions, longest, st);
-  if (mt == 2) return seql::launch<2>(p, n_portions, longest, st);
-  return seql::launch<1>(p, n_portions, longest, st);
+  mrs_seq_latent_attention_args a = {};
+  a.q = q; a.q_ld = q_ld; a.cache = cache; a.cache_row = cache_row; a.out = out; a.out_ld = out_ld;
+  a.portions = portions; a.cu_tok = cu_tok; a.past = past; a.n_portions = n_portions; a.longest = longest;
+  a.pages = pages; a.pages_ld = pages_ld; a.page_size = page_size; a.heads = heads; a.kv_rank = kv_rank; a.rot_dim = rot_dim;
+  a.scale = scale; a.window = window;
+  return mrs_seq_latent_attention_general(&a, stream);
 }

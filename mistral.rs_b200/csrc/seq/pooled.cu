@@ -86,6 +86,24 @@ __global__ void gate_cols_kernel(T *__restrict__ x, int64_t x_ld, const T *__res
   }
 }
 
+// four neighbouring entries per thread; all four share a gate when group is a multiple of four
+template <typename T>
+__global__ void gate_cols_vec_kernel(T *__restrict__ x, int64_t x_ld, const T *__restrict__ gate, int64_t gate_ld, int cols, int group, int act) {
+  const int t = blockIdx.x;
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4; c < cols; c += gridDim.y * blockDim.x * 4) {
+    float4 g;
+    if (group == 1) {
+      g = act4(load4<T>(gate + (int64_t)t * gate_ld + c), act);
+    } else {
+      const float one = apply_act(to_f32<T>(gate[(int64_t)t * gate_ld + c / group]), act);
+      g = make_float4(one, one, one, one);
+    }
+    T *at = x + (int64_t)t * x_ld + c;
+    const float4 v = load4<T>(at);
+    store4<T>(at, make_float4(v.x * g.x, v.y * g.y, v.z * g.z, v.w * g.w));
+  }
+}
+
 }  // namespace seq
 
 using namespace seq;
@@ -123,6 +141,14 @@ extern "C" int mrs_seq_gate_cols(void *x, int64_t x_ld, const void *gate, int64_
                                  int64_t stream) {
   if (n_tok <= 0 || cols <= 0) return 0;
   if (!x || !gate || group <= 0) return -2;
+  const int elem = dtype == MRS_SEQ_BF16 ? 2 : 4;
+  if (cols % 4 == 0 && x_ld % 4 == 0 && (uintptr_t)x % (4 * elem) == 0 &&
+      (group == 1 ? gate_ld % 4 == 0 && (uintptr_t)gate % (4 * elem) == 0 : group % 4 == 0)) {
+    const int vby = (cols / 4 + 255) / 256, vth = cols / 4 >= 256 ? 256 : 64;
+    SEQ_DISPATCH_DTYPE(dtype, (gate_cols_vec_kernel<T><<<dim3(n_tok, vby < 64 ? vby : 64), vth, 0, (cudaStream_t)stream>>>(
+                                  (T *)x, x_ld, (const T *)gate, gate_ld, cols, group, act)));
+    return launch_status();
+  }
   const int by = (cols + 255) / 256;
   SEQ_DISPATCH_DTYPE(dtype, (gate_cols_kernel<T><<<dim3(n_tok, by < 64 ? by : 64), 256, 0, (cudaStream_t)stream>>>(
                                 (T *)x, x_ld, (const T *)gate, gate_ld, cols, group, act)));

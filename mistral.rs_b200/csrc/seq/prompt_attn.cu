@@ -17,7 +17,7 @@
 // heads is then a weighted sum of these rows (pooled.cu's mix_heads).
 #include "../mma_common.cuh"
 
-#include "../../../include/mrs_b200_seq.h"
+#include "seq_common.cuh"
 
 namespace seqp {
 using namespace mrs;
@@ -39,6 +39,9 @@ struct Params {
   int64_t pool_base;
   int chunk;                   // > 0: a query sees only keys of its own chunk of positions
   int v_heads;                 // 1, or the number of value heads when every head is applied to every value head
+  const __nv_bfloat16 *gate;   // output gate per entry (gate_group 1) or per head (D); NULL: none
+  int64_t gate_ld;
+  int gate_group, gate_act;
   int o_f32;                   // the result is f32 [tokens, heads, v_heads * D] (o is then float *)
 };
 
@@ -235,8 +238,17 @@ __global__ void __launch_bounds__(THREADS, 1) prompt_attention_kernel(const Para
       if (row_a + 8 < len) *(float2 *)(ogf + (int64_t)(row_a + 8) * p.o_ld + col) = make_float2(oacc[i][2] * inv1, oacc[i][3] * inv1);
       continue;
     }
-    if (row_a < len) *(uint32_t *)(og + (int64_t)row_a * p.o_ld + col) = pack2<T>(oacc[i][0] * inv0, oacc[i][1] * inv0);
-    if (row_a + 8 < len) *(uint32_t *)(og + (int64_t)(row_a + 8) * p.o_ld + col) = pack2<T>(oacc[i][2] * inv1, oacc[i][3] * inv1);
+    float g[4] = {inv0, inv0, inv1, inv1};
+    if (p.gate) {
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int row = row_a + ((e >> 1) << 3);
+        if (row < len)
+          g[e] *= seq::apply_act(__bfloat162float(p.gate[(int64_t)(seq0 + row) * p.gate_ld + (h * D + col + (e & 1)) / p.gate_group]), p.gate_act);
+      }
+    }
+    if (row_a < len) *(uint32_t *)(og + (int64_t)row_a * p.o_ld + col) = pack2<T>(oacc[i][0] * g[0], oacc[i][1] * g[1]);
+    if (row_a + 8 < len) *(uint32_t *)(og + (int64_t)(row_a + 8) * p.o_ld + col) = pack2<T>(oacc[i][2] * g[2], oacc[i][3] * g[3]);
   }
 }
 
@@ -271,6 +283,7 @@ extern "C" int mrs_seq_prompt_attention_general(const mrs_seq_prompt_attention_a
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || (d != 64 && d != 128) || !a.portions || !a.pages || a.page_size <= 0) return -2;
   if (pool > 0 && (a.window <= 0 || a.keep_first > 0)) return -2;
   if (chunk > 0 && (a.keep_first > 0 || pool > 0)) return -2;
+  if (a.gate && (a.every_value_head || (a.gate_group != 1 && a.gate_group != d))) return -2;
   if ((int64_t)heads * (a.every_value_head ? kv_heads : 1) > 65535) return -2;
   if ((a.q_ld | a.out_ld) % 8 || (((uintptr_t)a.q | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache | (uintptr_t)a.out) & 15)) return -3;
   seqp::Params p = {};
@@ -282,6 +295,7 @@ extern "C" int mrs_seq_prompt_attention_general(const mrs_seq_prompt_attention_a
   p.window = a.window; p.keep_first = a.keep_first > 0 ? a.keep_first : 0; p.sink = a.sink;
   p.pool = pool; p.per_page = pool > 0 ? (a.page_size + pool - 1) / pool : 0; p.pool_base = a.pool_base;
   p.chunk = chunk;
+  p.gate = (const __nv_bfloat16 *)a.gate; p.gate_ld = a.gate_ld; p.gate_group = a.gate_group; p.gate_act = a.gate_act;
   p.v_heads = a.every_value_head ? kv_heads : 1;
   p.o_f32 = a.every_value_head ? 1 : 0;
   return d == 128 ? seqp::launch<128>(p, a.n_portions, a.longest, (cudaStream_t)stream)

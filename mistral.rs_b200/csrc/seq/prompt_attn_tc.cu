@@ -1,0 +1,404 @@
+// prompt_attn_tc.cu — causal prompt attention on the 5th-gen tensor cores (tcgen05 + TMEM) over DENSE keys and values, for
+// pieces of sequences that may continue: a segment is a run of query rows whose keys are dense rows k_row0 .. of which the
+// first `past` lie before its first query.  Keys are given head by head, optionally followed by ONE further part that all
+// heads share (the rotated part of a latent attention layer), so a head's score is q[0:dn] . k_h + q[dn:dn+dr] . k_shared;
+// value heads may have another size than key heads.  Callers bring whole prompts (keys straight from the projection), chunks
+// of a chunked layer (each its own segment, nothing to mask but the diagonal), or cached rows gathered / decompressed for the
+// step.
+//
+// One CTA = 128 query rows of one (segment, head), key tiles of BN rows, 192 threads (the roles of prefill_attn_tc.cu):
+//   warp 0      TMA: Q once, then K and V tiles, in SWIZZLE_128B boxes of 64 columns;
+//   warp 1      MMA issuer: S = Q K^T (both K-major in shared memory; 16 columns per MMA, dn / 16 + ceil(dr / 16) of them),
+//               O += P V (P in tensor memory, V from its row-major tile as an MN-major operand);
+//   warps 2..5  softmax + correction + epilogue, thread = query row = TMEM lane; P overwrites the head of S.
+// Two CTAs share an SM (one tile's softmax runs beside the other's products): BN is 128 while the tiles allow it, 64 with
+// three key boxes.  Boxes are always 64 columns wide.  Head sizes that do not fill their last box leave neighbouring columns
+// in it; the MMAs of S stop at the head's own columns (the shared part's box is filled with zeros past its end), and columns of
+// O past dv are never stored.
+//
+// Every wait has a limit; a wait that runs out sets a device flag (mrs_seq_prompt_attention_tc_timeouts) and ends the CTA.
+#include "../tc_common.cuh"
+
+#include "seq_common.cuh"
+
+namespace seqtc {
+using namespace mrs;
+
+constexpr int BM = 128, THREADS = 192;
+constexpr uint32_t TCOLS = 256, O_COL = 128, WAIT_LIMIT = 1u << 22;
+
+struct Params {
+  __nv_bfloat16 *o;
+  int64_t o_ld;
+  const int32_t *segments;     // [n][4]: first query row, query rows, first dense key row, keys before the first query
+  int H, KVH, dn, dr, dv;
+  float scale_log2;
+  const __nv_bfloat16 *gate;   // optional: result *= act(gate[row][(h * dv + d) / gate_group])
+  int64_t gate_ld;
+  int gate_group, gate_act;
+};
+
+__device__ int g_timeouts = 0;
+
+__device__ __forceinline__ bool wait_limited(uint64_t *bar, uint32_t parity) {
+  for (uint32_t i = 0; i < WAIT_LIMIT; i++) {
+    uint32_t done;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+        : "=r"(done)
+        : "r"(smem_u32(bar)), "r"(parity)
+        : "memory");
+    if (done) return true;
+  }
+  atomicExch(&g_timeouts, 1);
+  return false;
+}
+// shared-memory operand descriptor, SWIZZLE_128B, explicit leading / stride byte offsets
+__device__ __forceinline__ uint64_t desc_sw128_ex(uint32_t saddr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
+  const uint64_t addr = (uint64_t)(saddr >> 4) & 0x3FFF;
+  return addr | ((uint64_t)((lbo_bytes >> 4) & 0x3FFF) << 16) | ((uint64_t)((sbo_bytes >> 4) & 0x3FFF) << 32) | (1ull << 46) | (2ull << 61);
+}
+__device__ __forceinline__ void umma_ss_warp(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, e;\n\telect.sync _|e, 0xffffffff;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(tmem_d),
+      "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void tmem_ld_nowait(uint32_t taddr, uint32_t *r) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
+      "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
+        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
+        "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
+        "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+      : "r"(taddr));
+}
+__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const uint32_t *r) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::
+          "r"(taddr),
+      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
+      "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+      : "memory");
+}
+
+// NB: 64-column boxes of a head's own key columns; SH: 1 when a shared key part follows; NV: 64-column boxes of the values
+template <int NB, int SH, int NV> struct Shape {
+  static constexpr int BOXES = NB + SH, BN = BOXES > 2 ? 64 : 128;
+  static constexpr int QBOX = BM * 128, KBOX = BN * 128;                      // bytes of one box
+  static constexpr int Q_BYTES = BOXES * QBOX, K_BYTES = BOXES * KBOX, V_BYTES = NV * KBOX;
+  static constexpr int SMEM = 1024 + Q_BYTES + K_BYTES + V_BYTES + 256;
+};
+
+template <int NB, int SH, int NV>
+__global__ void __launch_bounds__(THREADS, 2)
+prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
+                           const __grid_constant__ CUtensorMap tmap_ks, const __grid_constant__ CUtensorMap tmap_v, const Params p) {
+  using S = Shape<NB, SH, NV>;
+  constexpr int BN = S::BN;
+  extern __shared__ __align__(1024) uint8_t smem_raw[];
+  uint8_t *smem = (uint8_t *)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint8_t *q_s = smem, *k_s = q_s + S::Q_BYTES, *v_s = k_s + S::K_BYTES;
+  uint64_t *bars = (uint64_t *)(v_s + S::V_BYTES);
+  uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 2, *v_full = bars + 3, *v_empty = bars + 4, *s_full = bars + 5,
+           *p_full = bars + 6, *pv_done = bars + 7;
+  uint32_t *tmem_slot = (uint32_t *)(bars + 8);
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, kvh = h / (p.H / p.KVH);
+  const int32_t *seg = p.segments + 4 * blockIdx.z;
+  const int row0 = seg[0], len = seg[1], key0 = seg[2], past = seg[3];
+  const int qt = (len + BM - 1) / BM - 1 - (int)blockIdx.x;          // heavy (late) query tiles first
+  if (qt < 0) return;
+  const int q0 = qt * BM;
+  const int kv_end = past + min(len, q0 + BM);
+  const int nt = (kv_end + BN - 1) / BN;                             // >= 1
+
+  if (warp == 0 && lane < 8) {
+    mbar_init(&bars[lane], lane == 6 ? 4u : 1u);                     // p_full: the four softmax warps
+    fence_mbar_init();
+  }
+  if (warp == 1) tmem_alloc(tmem_slot, TCOLS);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = __reduce_max_sync(0xffffffffu, *tmem_slot);
+  const uint32_t t_s = tmem_base, t_p = tmem_base, t_o = tmem_base + O_COL;      // P overwrites the head of S
+
+  if (warp == 0) {
+    // ===================== TMA producer =====================
+    const int qx = h * (p.dn + p.dr);
+    mbar_arrive_expect_tx_warp(q_full, S::Q_BYTES);
+#pragma unroll
+    for (int i = 0; i < NB; i++) tma_load_2d_warp(q_s + i * S::QBOX, &tmap_q, qx + 64 * i, row0 + q0, q_full);
+    if (SH) tma_load_2d_warp(q_s + NB * S::QBOX, &tmap_q, qx + p.dn, row0 + q0, q_full);
+    int k_issued = 0, v_issued = 0;
+    for (int j = 0; j < nt; j++) {
+      const int ph = j & 1, row = key0 + j * BN;
+      if (!wait_limited(k_empty, ph ^ 1)) break;
+      mbar_arrive_expect_tx_warp(k_full, S::K_BYTES);
+#pragma unroll
+      for (int i = 0; i < NB; i++) tma_load_2d_warp(k_s + i * S::KBOX, &tmap_k, kvh * p.dn + 64 * i, row, k_full);
+      if (SH) tma_load_2d_warp(k_s + NB * S::KBOX, &tmap_ks, 0, row, k_full);
+      k_issued = j + 1;
+      if (!wait_limited(v_empty, ph ^ 1)) break;
+      mbar_arrive_expect_tx_warp(v_full, S::V_BYTES);
+#pragma unroll
+      for (int i = 0; i < NV; i++) tma_load_2d_warp(v_s + i * S::KBOX, &tmap_v, kvh * p.dv + 64 * i, row, v_full);
+      v_issued = j + 1;
+    }
+    if (v_issued < nt) {                 // gave up: let the copies in flight land before the CTA may end
+      wait_limited(q_full, 0);
+      if (k_issued > 0) wait_limited(k_full, (k_issued - 1) & 1);
+      if (v_issued > 0) wait_limited(v_full, (v_issued - 1) & 1);
+    }
+  } else if (warp == 1) {
+    // ===================== MMA issuer =====================
+    // c = f32 (bit 4), a / b = bf16 (bits 7, 10), b_major = MN (bit 16) for the PV product, N >> 3 at bit 17, M >> 4 at bit 24
+    const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
+    const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(NV * 64 >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
+    const int own_steps = p.dn >> 4, shared_steps = SH ? (p.dr + 15) >> 4 : 0;
+    bool ok = wait_limited(q_full, 0);
+    int done = 0;                        // PV products committed
+    for (int j = 0; ok && j < nt; j++) {
+      const int ph = j & 1;
+      ok = wait_limited(k_full, ph);
+      if (ok && j > 0) ok = wait_limited(pv_done, ph ^ 1);           // PV_{j-1} has read P out of the S columns S_j overwrites
+      if (!ok) break;
+      tc_fence_after();
+      for (int c = 0; c < own_steps + shared_steps; c++) {
+        const int box = c < own_steps ? c >> 2 : NB, step = c < own_steps ? c & 3 : c - own_steps;
+        const uint64_t ad = umma_desc_sw128(q_s + box * S::QBOX) + (uint64_t)(2 * step);
+        const uint64_t bd = umma_desc_sw128(k_s + box * S::KBOX) + (uint64_t)(2 * step);
+        umma_ss_warp(t_s, ad, bd, idesc_s, c ? 1u : 0u);
+      }
+      umma_commit_warp(s_full);
+      umma_commit_warp(k_empty);
+      ok = wait_limited(p_full, ph) && wait_limited(v_full, ph);
+      if (!ok) break;
+      tc_fence_after();
+      const uint32_t vs = smem_u32(v_s);
+#pragma unroll
+      for (int c = 0; c < BN / 16; c++)   // 16 keys per MMA: two 8-row groups of 1024 B; the next 64 columns one box further
+        umma_f16_ts_warp(t_o, t_p + (uint32_t)(8 * c), desc_sw128_ex(vs + (uint32_t)c * 2048u, S::KBOX, 1024u), idesc_o, (j | c) ? 1u : 0u);
+      umma_commit_warp(pv_done);
+      umma_commit_warp(v_empty);
+      done = j + 1;
+    }
+    if (done > 0) wait_limited(pv_done, (done - 1) & 1);             // no product is in flight when tensor memory is freed
+  } else {
+    // ===================== softmax / correction / epilogue: thread = query row =====================
+    const int q4 = warp & 3, r = q4 * 32 + lane;
+    const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
+    const int qrow = q0 + r, qpos = past + qrow;                     // row inside the segment, position among its keys
+    // m_ref: the exponent's reference point; it moves only when a row's maximum outgrows it by more than 2^8 (then O and l
+    // are rescaled), so P lives in [0, 256] and the O round trip through tensor memory almost never happens
+    float m_ref = -INFINITY, l_run = 0.f;
+    bool ok = true;
+    for (int j = 0; ok && j < nt; j++) {
+      const int ph = j & 1;
+      const uint32_t ts = t_s + lane_off;
+      const int lim = min(qpos, kv_end - 1) - j * BN;                // columns > lim are masked
+      ok = wait_limited(s_full, ph);
+      if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+      tc_fence_after();
+      uint32_t v[BN];
+#pragma unroll
+      for (int c0 = 0; c0 < BN; c0 += 32) tmem_ld_nowait(ts + (uint32_t)c0, v + c0);
+      tmem_ld_wait();
+      float mx = -INFINITY;
+      if (lim >= BN - 1) {
+#pragma unroll
+        for (int i = 0; i < BN; i++) mx = fmaxf(mx, __uint_as_float(v[i]));
+      } else {
+#pragma unroll
+        for (int i = 0; i < BN; i++) {
+          if (i > lim) v[i] = 0xff800000u;                           // -inf: exp2 gives 0 below
+          mx = fmaxf(mx, __uint_as_float(v[i]));
+        }
+      }
+      mx *= p.scale_log2;                                            // (scale > 0: max commutes with the scaling)
+      const bool move = (m_ref == -INFINITY) || (mx > m_ref + 8.0f);
+      const float m_use = move ? fmaxf(m_ref, mx) : m_ref;
+      const float corr = (m_use == m_ref) ? 1.f : ex2(m_ref - m_use);
+      const float msub = (m_use == -INFINITY) ? 0.f : m_use;
+      if (j > 0 && __any_sync(0xffffffffu, corr != 1.f)) {           // PV_{j-1} is complete: S_j was issued after it
+#pragma unroll 1
+        for (int c0 = 0; c0 < NV * 64; c0 += 32) {
+          uint32_t o[32];
+          tmem_ld_32x32(t_o + lane_off + (uint32_t)c0, o);
+#pragma unroll
+          for (int i = 0; i < 32; i++) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr);
+          tmem_st_32x32(t_o + lane_off + (uint32_t)c0, o);
+        }
+      }
+      float rs = 0.f;
+#pragma unroll
+      for (int c0 = 0; c0 < BN; c0 += 32) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          const float p0 = ex2(fmaf(__uint_as_float(v[c0 + i]), p.scale_log2, -msub));
+          const float p1 = ex2(fmaf(__uint_as_float(v[c0 + i + 1]), p.scale_log2, -msub));
+          rs += p0 + p1;
+          const __nv_bfloat162 hh = __floats2bfloat162_rn(p0, p1);
+          pk[i >> 1] = *(const uint32_t *)&hh;
+        }
+        tmem_st_x16(t_p + lane_off + (uint32_t)(c0 >> 1), pk);
+      }
+      l_run = l_run * corr + rs;
+      m_ref = m_use;
+      tmem_wait_st();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full);
+    }
+    if (ok) ok = __all_sync(0xffffffffu, wait_limited(pv_done, (nt - 1) & 1));
+    if (ok) {                             // O / l -> global, times the output gate
+      tc_fence_after();
+      const float inv = (l_run > 0.f) ? 1.f / l_run : 0.f;
+      const int64_t row = row0 + qrow;
+      __nv_bfloat16 *orow = p.o + row * p.o_ld + (int64_t)h * p.dv;
+      const __nv_bfloat16 *grow = p.gate ? p.gate + row * p.gate_ld : nullptr;
+      const bool stores = qrow < len;
+      float head_gate = 1.f;
+      if (stores && grow && p.gate_group == p.dv) head_gate = seq::apply_act(__bfloat162float(grow[h]), p.gate_act);
+#pragma unroll 1
+      for (int c0 = 0; c0 < NV * 64; c0 += 32) {
+        uint32_t v[32];
+        tmem_ld_32x32(t_o + lane_off + (uint32_t)c0, v);
+        if (!stores) continue;
+#pragma unroll
+        for (int i = 0; i < 32; i += 8) {
+          if (c0 + i >= p.dv) break;
+          float x[8];
+#pragma unroll
+          for (int k = 0; k < 8; k++) x[k] = __uint_as_float(v[i + k]) * inv * head_gate;
+          if (grow && p.gate_group == 1) {
+            const uint4 raw = *(const uint4 *)(grow + (int64_t)h * p.dv + c0 + i);
+            const __nv_bfloat162 *g2 = (const __nv_bfloat162 *)&raw;
+#pragma unroll
+            for (int k = 0; k < 4; k++) {
+              const float2 g = __bfloat1622float2(g2[k]);
+              x[2 * k] *= seq::apply_act(g.x, p.gate_act);
+              x[2 * k + 1] *= seq::apply_act(g.y, p.gate_act);
+            }
+          }
+          uint4 pk;
+          uint32_t *w = (uint32_t *)&pk;
+#pragma unroll
+          for (int k = 0; k < 4; k++) {
+            const __nv_bfloat162 hh = __floats2bfloat162_rn(x[2 * k], x[2 * k + 1]);
+            w[k] = *(const uint32_t *)&hh;
+          }
+          *(uint4 *)(orow + c0 + i) = pk;
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem_base, TCOLS);
+}
+
+template <int NB, int SH, int NV>
+static int launch(const CUtensorMap &tq, const CUtensorMap &tk, const CUtensorMap &ts, const CUtensorMap &tv, const Params &p, int n, int longest,
+                  cudaStream_t st) {
+  auto kern = prompt_attention_tc_kernel<NB, SH, NV>;
+  constexpr int bytes = Shape<NB, SH, NV>::SMEM;
+  static bool raised = false;
+  if (!raised) {
+    const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return (int)e;
+    raised = true;
+  }
+  kern<<<dim3((longest + BM - 1) / BM, p.H, n), THREADS, bytes, st>>>(tq, tk, ts, tv, p);
+  return (int)cudaGetLastError();
+}
+
+// 16-byte copies of cached rows into dense rows: one warp per row
+__global__ void gather_rows_kernel(const uint4 *__restrict__ cache, int64_t row16, int n16, const int32_t *__restrict__ runs, const int32_t *__restrict__ pages,
+                                   int pages_ld, int page_size, uint4 *__restrict__ out, int64_t out16) {
+  const int32_t *run = runs + 4 * blockIdx.y;          // table row, first position, count, first dense row
+  const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= run[2]) return;
+  const int pos = run[1] + r;
+  const int64_t slot = (int64_t)pages[(int64_t)run[0] * pages_ld + pos / page_size] * page_size + pos % page_size;
+  const uint4 *src = cache + slot * row16;
+  uint4 *dst = out + (int64_t)(run[3] + r) * out16;
+  for (int c = lane; c < n16; c += 32) dst[c] = src[c];
+}
+
+}  // namespace seqtc
+
+extern "C" int mrs_seq_prompt_attention_tc_fits(int dn, int dr, int dv) {
+  return dn >= 16 && dn % 16 == 0 && dn <= 128 && dr >= 0 && dr % 8 == 0 && dr <= 64 && dv >= 8 && dv % 8 == 0 && dv <= 128 ? 1 : 0;
+}
+
+extern "C" int mrs_seq_prompt_attention_tc_timeouts(void) {
+  int v = 0;
+  const cudaError_t e = cudaMemcpyFromSymbol(&v, seqtc::g_timeouts, sizeof(int));
+  return e == cudaSuccess ? v : -(int)e;
+}
+
+extern "C" int mrs_seq_prompt_attention_tc(const mrs_seq_prompt_attention_tc_args *args, int64_t stream) {
+  using namespace seqtc;
+  const mrs_seq_prompt_attention_tc_args &a = *args;
+  if (a.n_segments <= 0 || a.longest <= 0) return 0;
+  if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.heads > 65535 || a.n_segments > 65535 || !a.segments || a.q_rows <= 0 || a.k_rows <= 0)
+    return -2;
+  if (!mrs_seq_prompt_attention_tc_fits(a.dn, a.dr, a.dv) || a.scale <= 0.0f || (a.dr > 0 && !a.k_shared)) return -2;
+  if (a.gate && a.gate_group != 1 && a.gate_group != a.dv) return -2;
+  auto al = [](const void *x) { return ((uintptr_t)x & 15) == 0; };
+  if ((a.q_ld | a.k_ld | a.v_ld | a.out_ld) % 8 || !al(a.q) || !al(a.k) || !al(a.v) || !al(a.out)) return -3;
+  if (a.dr > 0 && (a.k_shared_ld % 8 || !al(a.k_shared))) return -3;
+  if (a.gate && a.gate_group == 1 && (a.gate_ld % 8 || !al(a.gate))) return -3;
+  PFN_encodeTiled enc = tc_get_encode();
+  if (!enc) return -4;
+  const int nb = (a.dn + 63) / 64, sh = a.dr > 0 ? 1 : 0, nv = (a.dv + 63) / 64, bn = nb + sh > 2 ? 64 : 128;
+  auto make = [&](CUtensorMap *m, const void *base, int64_t cols, int64_t rows, int64_t ld, int box_rows) -> bool {
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {64u, (cuuint32_t)box_rows};
+    const cuuint32_t estr[2] = {1, 1};
+    return enc(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+  };
+  CUtensorMap tq, tk, ts, tv;
+  if (!make(&tq, a.q, (int64_t)a.heads * (a.dn + a.dr), a.q_rows, a.q_ld, BM) || !make(&tk, a.k, (int64_t)a.kv_heads * a.dn, a.k_rows, a.k_ld, bn) ||
+      !make(&tv, a.v, (int64_t)a.kv_heads * a.dv, a.k_rows, a.v_ld, bn))
+    return -4;
+  ts = tk;
+  if (sh && !make(&ts, a.k_shared, a.dr, a.k_rows, a.k_shared_ld, bn)) return -4;
+  Params p = {};
+  p.o = (__nv_bfloat16 *)a.out; p.o_ld = a.out_ld; p.segments = a.segments;
+  p.H = a.heads; p.KVH = a.kv_heads; p.dn = a.dn; p.dr = a.dr; p.dv = a.dv;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.gate = (const __nv_bfloat16 *)a.gate; p.gate_ld = a.gate_ld; p.gate_group = a.gate_group; p.gate_act = a.gate_act;
+  cudaStream_t st = (cudaStream_t)stream;
+#define SEQ_TC(NB, SH, NV) \
+  if (nb == NB && sh == SH && nv == NV) return launch<NB, SH, NV>(tq, tk, ts, tv, p, a.n_segments, a.longest, st)
+  SEQ_TC(1, 0, 1); SEQ_TC(1, 0, 2); SEQ_TC(1, 1, 1); SEQ_TC(1, 1, 2);
+  SEQ_TC(2, 0, 1); SEQ_TC(2, 0, 2); SEQ_TC(2, 1, 1); SEQ_TC(2, 1, 2);
+#undef SEQ_TC
+  return -2;
+}
+
+extern "C" int mrs_seq_gather_rows(const void *cache, int64_t cache_row_bytes, int row_bytes, const int32_t *runs, int n_runs, int longest,
+                                   const int32_t *pages, int pages_ld, int page_size, void *out, int64_t out_row_bytes, int64_t stream) {
+  if (n_runs <= 0 || longest <= 0) return 0;
+  if (!cache || !runs || !pages || !out || page_size <= 0 || n_runs > 65535) return -2;
+  if ((cache_row_bytes | out_row_bytes | row_bytes) % 16 || (((uintptr_t)cache | (uintptr_t)out) & 15)) return -3;
+  seqtc::gather_rows_kernel<<<dim3((longest + 7) / 8, n_runs), 256, 0, (cudaStream_t)stream>>>(
+      (const uint4 *)cache, cache_row_bytes / 16, row_bytes / 16, runs, pages, pages_ld, page_size, (uint4 *)out, out_row_bytes / 16);
+  return (int)cudaGetLastError();
+}

@@ -104,6 +104,10 @@ __device__ __forceinline__ int64_t key_row(const int32_t *table, int j, int pool
   const int page = (j * pool) / page_size, first = (page * page_size + pool - 1) / pool;
   return pool_base + (int64_t)table[page] * per_page + (j - first);
 }
+// The output gate of entry c of a token's concatenated heads (1 without a gate)
+template <typename T> __device__ __forceinline__ float out_gate(const T *gate, int64_t gate_ld, int t, int c, int group, int act) {
+  return gate ? apply_act(to_f32<T>(gate[(int64_t)t * gate_ld + c / group]), act) : 1.0f;
+}
 // First position a query sees through a sliding window and / or through chunks counted from position 0
 __device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
   int lo = window > 0 ? max(0, pos - window + 1) : 0;
@@ -127,7 +131,7 @@ __global__ void __launch_bounds__(128) window_attention_kernel(const T *__restri
                                                                const int32_t *__restrict__ pos_of_tok, const int32_t *__restrict__ tok_index,
                                                                int n_tok, T *__restrict__ out, int64_t out_ld, float out_scale, int64_t k_row,
                                                                int64_t v_row, int pool, int64_t pool_base, int v_shared, int out_f32, int64_t out_head,
-    int chunk) {
+    int chunk, const T *__restrict__ gate, int64_t gate_ld, int gate_group, int gate_act) {
   extern __shared__ __align__(16) float qsm[];   // [warps][dk]
   const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
   const int64_t job = (int64_t)blockIdx.x * (blockDim.x >> 5) + wib;
@@ -184,7 +188,9 @@ __global__ void __launch_bounds__(128) window_attention_kernel(const T *__restri
   const float inv = out_scale / l;
 #pragma unroll
   for (int c = 0; c < MAX_VCOLS; c++)
-    if (c * 32 + lane < dv) store_out<T>(out, (int64_t)t * out_ld + h * out_head + c * 32 + lane, acc[c] * inv, out_f32);
+    if (c * 32 + lane < dv)
+      store_out<T>(out, (int64_t)t * out_ld + h * out_head + c * 32 + lane,
+                   acc[c] * inv * out_gate<T>(gate, gate_ld, t, h * dv + c * 32 + lane, gate_group, gate_act), out_f32);
 }
 
 // The same computation laid out for speed when the head sizes allow vector loads (dk a multiple of 8 and dv even):
@@ -197,7 +203,7 @@ __global__ void __launch_bounds__(SPLIT * 32) window_attention_vec_kernel(
     float scale, int window, int keep_first, const float *__restrict__ sink, const int32_t *__restrict__ pages, int pages_ld, int page_size,
     const int32_t *__restrict__ seq_of_tok, const int32_t *__restrict__ pos_of_tok, const int32_t *__restrict__ tok_index, T *__restrict__ out,
     int64_t out_ld, float out_scale, int64_t k_row, int64_t v_row, int pool, int64_t pool_base, int v_shared, int out_f32, int64_t out_head,
-    int chunk) {
+    int chunk, const T *__restrict__ gate, int64_t gate_ld, int gate_group, int gate_act) {
   extern __shared__ __align__(16) float sm[];   // q [dk] | per warp: m, l, acc [VPAIRS * 64]
   const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
   const int ti = blockIdx.x / heads, h = blockIdx.x % heads, t = tok_index ? tok_index[ti] : ti, g = h / (heads / kv_heads);
@@ -288,7 +294,7 @@ __global__ void __launch_bounds__(SPLIT * 32) window_attention_vec_kernel(
       const float mw = part[w * (2 + VPAIRS * 64)];
       if (mw != -INFINITY) o = fmaf(part[w * (2 + VPAIRS * 64) + 2 + c], expf(mw - mx), o);
     }
-    store_out<T>(out, (int64_t)t * out_ld + h * out_head + c, o * inv, out_f32);
+    store_out<T>(out, (int64_t)t * out_ld + h * out_head + c, o * inv * out_gate<T>(gate, gate_ld, t, h * dv + c, gate_group, gate_act), out_f32);
   }
 }
 
@@ -344,6 +350,7 @@ extern "C" int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args,
   const int keep_first = a.keep_first > 0 ? a.keep_first : 0, pool = a.pool > 0 ? a.pool : 0;
   if (pool > 0 && (a.window <= 0 || keep_first > 0)) return -2;      // averaged blocks lie before a window and replace kept first keys
   const int chunk = a.chunk > 0 ? a.chunk : 0;
+  if (a.gate && (a.v_shared || (a.gate_group != 1 && a.gate_group != dv))) return -2;
   if (chunk > 0 && (keep_first > 0 || pool > 0)) return -2;          // what lies before the chunk is not seen
   cudaStream_t st = (cudaStream_t)stream;
   const int elem = dtype == MRS_SEQ_BF16 ? 2 : 4;
@@ -357,7 +364,7 @@ extern "C" int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args,
   window_attention_vec_kernel<T, VP, SPLIT><<<(unsigned)n_tok * heads, SPLIT * 32, (dk + SPLIT * (2 + VP * 64)) * sizeof(float), st>>>( \
       (const T *)a.q, a.q_ld, (const T *)a.k_cache, (const T *)a.v_cache, heads, kv_heads, dk, dv, a.scale, a.window, keep_first, a.sink,  \
       a.pages, a.pages_ld, a.page_size, a.seq_of_tok, a.pos_of_tok, a.tok_index, (T *)a.out, a.out_ld, a.out_scale, k_row, v_row, pool,     \
-      a.pool_base, a.v_shared, a.out_f32, out_head, chunk)
+      a.pool_base, a.v_shared, a.out_f32, out_head, chunk, (const T *)a.gate, a.gate_ld, a.gate_group, a.gate_act)
     SEQ_DISPATCH_DTYPE(dtype, {
       if (dv <= 64) SEQ_ATTN_VEC(1);
       else if (dv <= 128) SEQ_ATTN_VEC(2);
@@ -373,7 +380,7 @@ extern "C" int mrs_seq_paged_attention(const mrs_seq_paged_attention_args *args,
   window_attention_kernel<T, VC><<<(unsigned)((jobs + warps - 1) / warps), warps * 32, warps * dk * sizeof(float), st>>>(  \
       (const T *)a.q, a.q_ld, (const T *)a.k_cache, (const T *)a.v_cache, heads, kv_heads, dk, dv, a.scale, a.window, keep_first, a.sink, \
       a.pages, a.pages_ld, a.page_size, a.seq_of_tok, a.pos_of_tok, a.tok_index, n_tok, (T *)a.out, a.out_ld, a.out_scale, k_row, v_row, pool, \
-      a.pool_base, a.v_shared, a.out_f32, out_head, chunk)
+      a.pool_base, a.v_shared, a.out_f32, out_head, chunk, (const T *)a.gate, a.gate_ld, a.gate_group, a.gate_act)
   SEQ_DISPATCH_DTYPE(dtype, {
     if (dv <= 64) SEQ_ATTN_LAUNCH(2);
     else if (dv <= 128) SEQ_ATTN_LAUNCH(4);

@@ -103,7 +103,8 @@ class StepBatch:
         paged = np.concatenate([np.arange(cu[b], cu[b + 1], dtype=np.int32) for b in range(n_seq) if not is_fresh[b]] + [np.zeros(0, np.int32)])
         # long portions, fresh or continued: (first row, rows, tokens cached before, sequence) for kernels that tile a portion's rows
         is_long = [c >= self.FRESH_MIN for c in counts]
-        self.long = [(int(cu[b]), int(counts[b]), int(pasts[b]), b) for b in range(n_seq) if is_long[b]]
+        self.portions = [(int(cu[b]), int(counts[b]), int(pasts[b]), b) for b in range(n_seq)]
+        self.long = [p for p, yes in zip(self.portions, is_long) if yes]
         long_rows = np.asarray(self.long, dtype=np.int32).reshape(-1)
         short = np.concatenate([np.arange(cu[b], cu[b + 1], dtype=np.int32) for b in range(n_seq) if not is_long[b]] + [np.zeros(0, np.int32)])
         parts = [np.asarray(ids, dtype=np.int32), cu, np.asarray(pasts, dtype=np.int32), np.asarray(slots, dtype=np.int32), seq_of, pos_of,
@@ -136,6 +137,60 @@ class StepBatch:
         self.short_tok = cut(10)                                   # tokens of the sequences not in `long`
         at = int(o[-1]) + pad
         self.slot_of_tok = dev[at:at + 2 * n_tok].view(torch.int64)
+
+
+    def device_ints(self, values):
+        """A host list of integers as an int32 device tensor that lives as long as this batch (plans that mixers make per step)."""
+        host = torch.tensor(values, dtype=torch.int32)
+        host = host.pin_memory() if torch.cuda.is_available() else host
+        self.__dict__.setdefault("_held", []).append(host)
+        return host.to(self.device, non_blocking=True)
+
+    def dense_plan(self, min_rows, chunk):
+        """How the portions of at least `min_rows` tokens run over dense keys (`seq_ops.tc_attention`), one plan per step and rule:
+        every such portion is cut at the borders of its chunks (`chunk` 0: not cut), every piece is one segment whose keys start
+        at its chunk.  None when no portion is that long."""
+        plans = self.__dict__.setdefault("_dense_plans", {})
+        if (min_rows, chunk) not in plans:
+            plans[min_rows, chunk] = DensePlan(self, min_rows, chunk) if any(n >= min_rows for _, n, _, _ in self.portions) else None
+        return plans[min_rows, chunk]
+
+
+class DensePlan:
+    """See `StepBatch.dense_plan`.  `segments` index dense rows that `runs` (sequence, first position, positions, first dense row)
+    gather from the pages.  `own_segments`, None unless no piece has keys before its own first token: the same with the step's
+    own rows as dense rows, for keys and values taken straight from the step's projections.  `rest_rows` / `rest`: the step's
+    rows and portions (first row inside the compacted rest) outside the plan."""
+
+    def __init__(self, batch, min_rows, chunk):
+        taken = [p for p in batch.portions if p[1] >= min_rows]
+        pieces = []                                               # (first row, rows, sequence, chunk's first position, keys before)
+        for row0, n, past, b in taken:
+            at, end = past, past + n
+            while at < end:
+                lo = at // chunk * chunk if chunk > 0 else 0
+                stop = min(end, lo + chunk) if chunk > 0 else end
+                pieces.append((row0 + at - past, stop - at, b, lo, at - lo))
+                at = stop
+        segments, runs, self.n_rows = [], [], 0
+        for row, n, b, lo, before in pieces:
+            segments += [row, n, self.n_rows, before]
+            runs += [b, lo, before + n, self.n_rows]
+            self.n_rows += before + n
+        self.n, self.longest, self.longest_run = len(pieces), max(p[1] for p in pieces), max(p[4] + p[1] for p in pieces)
+        self.segments, self.runs = batch.device_ints(segments), batch.device_ints(runs)
+        fresh = all(before == 0 for *_, before in pieces)
+        self.own_segments = batch.device_ints([v for row, n, *_ in pieces for v in (row, n, row, 0)]) if fresh else None
+        self.rest, self.rest_rows, rows, at = [], None, [], 0
+        for row0, n, past, b in batch.portions:
+            if n < min_rows:
+                self.rest.append((at, n, past, b))
+                rows += range(row0, row0 + n)
+                at += n
+        if rows:
+            self.rest_rows = batch.device_ints(rows)
+            self.rest_portions = batch.device_ints([v for p in self.rest for v in p])
+            self.rest_longest = max(p[1] for p in self.rest)
 
 
 class DecodeGraph:

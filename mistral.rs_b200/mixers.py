@@ -174,13 +174,18 @@ class WindowAttention:
                gate_group=1):
         """y holds q | k | v (q | k when the values are the keys) from column col0; writes heads * dv columns of `out`
         from out_col.  Keys and values of the new tokens are normed, rotated and stored first.  Long portions (32 tokens
-        or more) run on tensor cores when they fit (bf16, equal head sizes of 64 or 128, 16-byte aligned rows): when every
-        one of them starts its sequence and the layer has neither sink nor kept first tokens, on the package's prompt
-        kernels over the fresh q / k / v; otherwise — sinks, kept tokens, portions that continue a sequence — on the
-        sequence library's prompt kernel, which reads keys and values from the pages.  Every other token (short portions,
-        decoded tokens, other head sizes, f32) runs on the (token, head) kernel over the pages, and so does every token of a
-        layer with averaged blocks or mixed heads.  gate_col: columns of y whose `gate_act` multiplies the result, one column per
-        `gate_group` neighbouring entries (1: entry by entry; dv: one number per head, not with mixed heads)."""
+        or more) run on tensor cores when they fit (bf16, 16-byte aligned rows):
+          * plain causal layers and layers with chunks (no window, sink or kept first tokens; head sizes `tc_attention` takes) on
+            the tcgen05 kernel over dense keys and values — the step's own projections when every piece starts its sequence or
+            chunk, otherwise rows gathered from the pages;
+          * equal head sizes of 64 or 128, a window, every portion starting its sequence, neither sink nor kept first tokens: the
+            package's prompt kernels over the fresh q / k / v;
+          * other layers of equal head sizes of 64 or 128 on the sequence library's mma.sync prompt kernel, which reads keys and
+            values from the pages.
+        Every other token (short portions, decoded tokens, other head sizes, f32) runs on the (token, head) kernel over the
+        pages, and so does every token of a layer with averaged blocks or mixed heads.  gate_col: columns of y whose `gate_act`
+        multiplies the result, one column per `gate_group` neighbouring entries (1: entry by entry; dv: one number per head, not
+        with mixed heads)."""
         kc = col0 + self.heads * self.dk
         vc = None if self.values_from_keys else kc + self.kv_heads * self.dk
         cos_sin = self.rotation.table(batch) if self.rotation is not None else None
@@ -194,9 +199,8 @@ class WindowAttention:
         if self.pool > 0 or self.talk is not None:
             self._attend_general(y, col0, batch, cache, page_size, out, out_col, out_scale, gate_col, gate_act, gate_group)
             return
-        self._attend_plain(y, col0, kc, vc, batch, cache, page_size, out, out_col, out_scale)
-        if gate_col is not None:
-            K.gate_cols(out[:, out_col:], y, gate_col, self.heads * self.dv, gate_group, gate_act)
+        gate = {} if gate_col is None else {"gate": y, "gate_col": gate_col, "gate_group": gate_group, "gate_act": gate_act}
+        self._attend_plain(y, col0, kc, vc, batch, cache, page_size, out, out_col, out_scale, gate)
 
     def _attend_general(self, y, col0, batch, cache, page_size, out, out_col, out_scale, gate_col, gate_act, gate_group):
         """Averaged blocks and / or mixed heads.  Long portions take the sequence library's tensor-core prompt kernel when they
@@ -234,25 +238,42 @@ class WindowAttention:
         elif gate_col is not None:
             K.gate_cols(out[:, out_col:], y, gate_col, H * dv, gate_group, gate_act)
 
-    def _attend_plain(self, y, col0, kc, vc, batch, cache, page_size, out, out_col, out_scale):
+    MIN_CHUNK = 64           # smaller chunks leave most of a 128-row query tile empty when each is a segment of its own
+
+    def _attend_plain(self, y, col0, kc, vc, batch, cache, page_size, out, out_col, out_scale, gate):
+        H, G, dk, dv = self.heads, self.kv_heads, self.dk, self.dv
         tok_index = None
-        aligned = all(v % 8 == 0 for v in (y.stride(0), col0, out.stride(0), out_col))
-        if batch.long and y.dtype == torch.bfloat16 and self.dk == self.dv and self.dk in (64, 128) and aligned:
-            plain = self.sink is None and self.keep_first == 0 and self.chunk == 0 and vc is not None       # what the package's prompt kernels know
-            if plain and len(batch.fresh) == len(batch.long):
-                for row0, rows in batch.fresh:
-                    K.fresh_prompt_attention(y, row0, rows, col0, kc, vc, self.heads, self.kv_heads, self.dk, self.scale, self.window, out, out_col)
+        aligned = y.dtype == torch.bfloat16 and all(v % 8 == 0 for v in (y.stride(0), col0, out.stride(0), out_col))
+        plain = self.sink is None and self.keep_first == 0 and vc is not None
+        if batch.long and aligned and plain and self.window <= 0 and (self.chunk == 0 or self.chunk >= self.MIN_CHUNK) and \
+                K.tc_attention_fits(dk, 0, dv, kc, vc, G * dk, G * dv, *((gate["gate_col"],) if gate and gate["gate_group"] == 1 else ())):
+            plan = batch.dense_plan(batch.FRESH_MIN, self.chunk)
+            if plan.own_segments is not None:
+                segments, k, k_col, v, v_col = plan.own_segments, y, kc, y, vc
             else:
-                K.prompt_attention(y, col0, cache["k"], cache["v"], batch, page_size, self.heads, self.kv_heads, self.dk, self.scale, self.window,
-                                   self.keep_first, self.sink, out, out_col, chunk=self.chunk)
+                segments = plan.segments
+                gather = lambda c: K.gather_rows(c.flatten(1), c.shape[1] * c.shape[2], plan.runs, plan.n, plan.longest_run, batch, page_size, plan.n_rows)
+                k, k_col, v, v_col = gather(cache["k"]), 0, gather(cache["v"]), 0
+            K.tc_attention(y, col0, k, k_col, v, v_col, segments, plan.n, plan.longest, H, G, dk, 0, dv, self.scale, out, out_col, **gate)
+            tok_index = batch.short_tok
+        elif batch.long and aligned and dk == dv and dk in (64, 128):
+            if plain and self.chunk == 0 and len(batch.fresh) == len(batch.long):       # what the package's prompt kernels know
+                for row0, rows in batch.fresh:
+                    K.fresh_prompt_attention(y, row0, rows, col0, kc, vc, H, G, dk, self.scale, self.window, out, out_col)
+                    if gate:
+                        K.gate_cols(out[row0:row0 + rows, out_col:], y[row0:row0 + rows], gate["gate_col"], H * dv, gate["gate_group"], gate["gate_act"])
+            else:
+                K.prompt_attention(y, col0, cache["k"], cache["v"], batch, page_size, H, G, dk, self.scale, self.window, self.keep_first, self.sink, out,
+                                   out_col, chunk=self.chunk, **gate)
+            tok_index = batch.short_tok
+        if tok_index is not None:
             if out_scale != 1.0:
                 for row0, rows, _, _ in batch.long:
-                    K.scale_rows(out, row0, rows, out_col, self.heads * self.dv, out_scale)
-            tok_index = batch.short_tok
+                    K.scale_rows(out, row0, rows, out_col, H * dv, out_scale)
             if tok_index.numel() == 0:
                 return
-        K.paged_attention(y, col0, cache["k"], cache["v"], self.heads, self.kv_heads, self.dk, self.dv, self.scale, self.window,
-                          self.keep_first, self.sink, batch, page_size, out, out_col, out_scale, tok_index, chunk=self.chunk)
+        K.paged_attention(y, col0, cache["k"], cache["v"], H, G, dk, dv, self.scale, self.window, self.keep_first, self.sink, batch, page_size, out,
+                          out_col, out_scale, tok_index, chunk=self.chunk, **gate)
 
 
 class InputConvolution:
@@ -295,10 +316,12 @@ class LatentAttentionMixer:
     tensor-core latent kernel (all heads of a token share one fetched key tile); f32, and sizes the kernel does not take,
     run on the (token, head) kernel over the pages.  `shares`: this mixer has no W_dkv and reads the cache another layer fills.
 
-    When every sequence of a step starts in it with a long portion (whole prompts) and the sizes allow (bf16, no rotated part,
-    dn = dv of 64 or 128, at least DECOMPRESS_MIN_TOKENS tokens), keys and values ARE decompressed, for this step only: two
-    products turn the step's normed latents into per-head keys and values, and the plain tensor-core prompt kernel runs over
-    these dense rows — dn + dv multiply-adds per (query, key, head) instead of 2 kv_rank.  The cache still holds only latents.
+    Long portions (`decompress_min` tokens or more, of a prompt's start or a later part of it) decompress keys and values, for
+    this step only, when the sizes allow (bf16, no window, head sizes `seq_ops.tc_attention` takes): the latents of everything
+    such a portion sees become dense rows — the step's own, or gathered from the pages — one product turns them into per-head
+    keys and values, and the tcgen05 prompt kernel runs over those, the rotated part as one further key part all heads share: dn +
+    dr + dv multiply-adds per (query, key, head) instead of 2 kv_rank + dr.  The cache holds only latents either way; the other
+    sequences of the step stay in the absorbed form.
 
     q_rank 0: there is no query latent — w_down's first heads * (dn + dr) rows are the query projection itself (w_uq and
     q_norm_w are None).  dr 0 with rotation None: no rotated part, scores carry no position.  `head_gate`: w_down ends with
@@ -312,9 +335,9 @@ class LatentAttentionMixer:
         self.gate_act, self.gate_group = (head_gate, dv) if head_gate is not None else (entry_gate, 1)
         self.pairing = pairing
         self.w_down, self.w_uq, self.w_o, self.q_norm_w, self.kv_norm_w = w_down, w_uq, w_o, q_norm_w, kv_norm_w
-        self.w_uk_rows, self.w_uv_rows = w_uk, w_uv                      # [H dn, r] / [H dv, r]: the decompressing products
-        self.w_uk = w_uk.view(heads, dn, kv_rank)                       # [H][dn][r]: q_plain,h @ w_uk[h] = W_uk,h^T q_plain,h
-        self.w_uv_t = w_uv.view(heads, dv, kv_rank).transpose(1, 2)     # [H][r][dv]
+        self.w_ukv = torch.cat([w_uk, w_uv]).contiguous()               # [H dn + H dv, r]: the decompressing product
+        self.w_uk = self.w_ukv[:heads * dn].view(heads, dn, kv_rank)    # [H][dn][r]: q_plain,h @ w_uk[h] = W_uk,h^T q_plain,h
+        self.w_uv_t = self.w_ukv[heads * dn:].view(heads, dv, kv_rank).transpose(1, 2)     # [H][r][dv]
         self.heads, self.dn, self.dr, self.dv, self.q_rank, self.kv_rank = heads, dn, dr, dv, q_rank, kv_rank
         self.scale, self.window, self.rotation, self.eps, self.page_size, self.shares = scale, window, rotation, eps, page_size, shares
         self.row = kv_rank + dr
@@ -325,60 +348,89 @@ class LatentAttentionMixer:
         row = -(-self.row // 8) * 8            # rows start on 16-byte boundaries
         return {"latent": torch.zeros(n_token_slots, row, dtype=dtype, device=device)}
 
-    DECOMPRESS_MIN_TOKENS = 256
+    DECOMPRESS_MIN_TOKENS = 64
+    DECOMPRESS_MAX_BYTES = 4 << 30        # of decompressed keys and values held for one layer of one step
 
-    def decompresses(self, h, batch):
-        """True when this step's keys and values are decompressed (see the class text)."""
-        return (h.dtype == torch.bfloat16 and not self.shares and self.dr == 0 and self.dn == self.dv and self.dv in (64, 128) and
-                self.kv_rank % 8 == 0 and self.w_down.shape[0] % 8 == 0 and batch.n_seq > 0 and len(batch.long) == batch.n_seq and
-                all(past == 0 for _, _, past, _ in batch.long) and h.shape[0] >= self.DECOMPRESS_MIN_TOKENS)
+    def decompress_plan(self, h, batch):
+        """The step's `engine.DensePlan` of portions whose keys and values are decompressed, or None.  Decompressing costs
+        kv_rank (dn + dv) multiply-adds per key and head, and saves 2 kv_rank - dn - dv per (query, key, head)."""
+        saved = 2 * self.kv_rank - self.dn - self.dv
+        if h.dtype != torch.bfloat16 or self.window > 0 or batch.longest < self.DECOMPRESS_MIN_TOKENS or saved <= 0 or \
+                not K.latent_attention_fits(self.kv_rank, self.dr):
+            return None
+        min_rows = max(self.DECOMPRESS_MIN_TOKENS, -(-self.kv_rank * (self.dn + self.dv) // (4 * saved)))
+        cols = self.heads * (self.dn + self.dv)
+        gate = () if self.gate_group != 1 or self.gate_act is None else (self.gate_col,)
+        if batch.longest < min_rows or not K.tc_attention_fits(self.dn, self.dr, self.dv, self.w_down.shape[0], self.heads * self.dn, cols, self.kv_rank,
+                                                               self.heads * self.dv, self.heads * (self.dn + self.dr), *gate):
+            return None
+        plan = batch.dense_plan(min_rows, 0)
+        return plan if plan is not None and plan.n_rows * cols * 2 <= self.DECOMPRESS_MAX_BYTES else None
+
+    @property
+    def q_cols(self):
+        return self.q_rank if self.q_rank > 0 else self.heads * (self.dn + self.dr)
+
+    @property
+    def gate_col(self):
+        """First gate column of the input projection's result."""
+        return self.q_cols + (0 if self.shares else self.kv_rank + self.dr)
 
     def forward(self, h, batch, cache):
-        T, H, dn, dr, R = h.shape[0], self.heads, self.dn, self.dr, self.kv_rank
-        latent = cache["latent"]
-        if self.decompresses(h, batch):
-            y = linear(h, self.w_down)
-            q_cols = self.q_rank if self.q_rank > 0 else H * dn
-            c = torch.empty(T, R, dtype=h.dtype, device=h.device)
-            cq = torch.empty(T, self.q_rank, dtype=h.dtype, device=h.device) if self.q_rank > 0 else None
-            K.latent_prepare(y, 0, self.q_rank, self.q_norm_w, cq, q_cols, R, 0, 0, self.kv_norm_w, None, self.eps, latent, batch.slot_of_tok, kv_out=c)
-            q2 = linear(cq, self.w_uq) if self.q_rank > 0 else y
-            out = torch.empty(T, H * self.dv, dtype=h.dtype, device=h.device)
-            K.dense_prompt_attention(q2, 0, linear(c, self.w_uk_rows), linear(c, self.w_uv_rows), batch, H, H, self.dv, self.scale, self.window,
-                                     None, out)
-            if self.gate_act is not None:
-                K.gate_cols(out, y, q_cols + R, H * self.dv, self.gate_group, self.gate_act)
-            return linear(out, self.w_o)
+        T, H, dn, dr, dv, R = h.shape[0], self.heads, self.dn, self.dr, self.dv, self.kv_rank
+        latent, plan = cache["latent"], self.decompress_plan(h, batch)
         cos_sin = self.rotation.table(batch) if self.rotation is not None else None
         rot_dims = self.rotation.dims if self.rotation is not None else 0
-        y = linear(h, self.w_down)                                           # query latent (or queries) | (key/value latent | shared key part) | (gates)
-        q_cols = self.q_rank if self.q_rank > 0 else H * (dn + dr)
-        if self.q_rank > 0:
-            cq = torch.empty(T, self.q_rank, dtype=h.dtype, device=h.device)
-            K.latent_prepare(y, 0, self.q_rank, self.q_norm_w, cq, q_cols, 0 if self.shares else R, dr, rot_dims, self.kv_norm_w, cos_sin,
-                             self.eps, latent, batch.slot_of_tok, pairing=self.pairing)
-            q2 = linear(cq, self.w_uq)
+        y = linear(h, self.w_down)                                # query latent (or queries) | (key/value latent | shared key part) | (gates)
+        # where the queries' rotated parts go: into the absorbed queries, or in place for the decompressed form
+        qa = torch.empty(T, H, self.row, dtype=h.dtype, device=h.device) if plan is None else None
+        own = plan is not None and plan.own_segments is not None and not self.shares         # the step's own latents are all it takes
+        dense = torch.empty(T, latent.shape[1], dtype=h.dtype, device=h.device) if own else None
+        turn = lambda src: (H, dn, dn + dr, src, dn, dn + dr) if plan is not None else (H, dn, dn + dr, qa.view(T, -1), R, self.row)
+        cq = torch.empty(T, self.q_rank, dtype=h.dtype, device=h.device) if self.q_rank > 0 else None
+        rotate_q = turn(y) if dr > 0 and self.q_rank == 0 else None
+        if not self.shares or self.q_rank > 0 or rotate_q is not None:
+            K.latent_prepare(y, 0, self.q_rank, self.q_norm_w, cq, self.q_cols, 0 if self.shares else R, dr, rot_dims, self.kv_norm_w, cos_sin,
+                             self.eps, latent, batch.slot_of_tok, kv_out=dense, pairing=self.pairing, rotate_q=rotate_q)
+        q2 = linear(cq, self.w_uq) if self.q_rank > 0 else y
+        if dr > 0 and self.q_rank > 0:
+            _, col, step, dst, dst_col, dst_step = turn(q2)
+            K.rotate_pairs(q2, col, step, dst, dst_col, dst_step, H, dr, rot_dims, cos_sin, pairing=self.pairing)
+        out = torch.empty(T, H * dv, dtype=h.dtype, device=h.device)
+        gated = {} if self.gate_act is None else {"gate": y, "gate_col": self.gate_col, "gate_group": self.gate_group, "gate_act": self.gate_act}
+        if plan is None:
+            self._absorbed(q2, qa, y, latent, batch, out)
         else:
-            if not self.shares:
-                K.latent_prepare(y, 0, 0, None, None, q_cols, R, dr, rot_dims, self.kv_norm_w, cos_sin, self.eps, latent, batch.slot_of_tok,
-                                 pairing=self.pairing)
-            q2 = y[:, :q_cols]
-        q = q2.unflatten(1, (H, dn + dr))
-        qa = torch.empty(T, H, self.row, dtype=h.dtype, device=h.device)      # the absorbed queries
+            if dense is None:                                    # rows of everything the long portions see
+                dense = K.gather_rows(latent, latent.shape[1], plan.runs, plan.n, plan.longest_run, batch, self.page_size, plan.n_rows)
+            kv = linear(dense[:, :R], self.w_ukv)                 # [rows, H dn | H dv]
+            K.tc_attention(q2, 0, kv, 0, kv, H * dn, plan.own_segments if own else plan.segments, plan.n, plan.longest, H, H, dn, dr, dv, self.scale, out, k_shared=dense,
+                           k_shared_col=R, **gated)
+            if plan.rest:                                        # short portions and decoded tokens of the same step, compacted
+                rows = plan.rest_rows
+                q_rest, out_rest = q2.index_select(0, rows), torch.empty(rows.numel(), H * dv, dtype=h.dtype, device=h.device)
+                qa = torch.empty(rows.numel(), H, self.row, dtype=h.dtype, device=h.device)
+                if dr > 0:
+                    qa[:, :, R:] = q_rest[:, :H * (dn + dr)].unflatten(1, (H, dn + dr))[:, :, dn:]
+                self._absorbed(q_rest, qa, y.index_select(0, rows) if self.gate_act is not None else None, latent, batch, out_rest, plan)
+                out.index_copy_(0, rows.long(), out_rest)
+        return linear(out, self.w_o)
+
+    def _absorbed(self, q2, qa, y, latent, batch, out, plan=None):
+        """Absorbed latent attention of the step's rows (or of `plan`'s rest): q2 holds the queries, qa their rotated parts already;
+        writes `out` [rows, H * dv], gated by columns of y."""
+        T, H, dn, dr, R = qa.shape[0], self.heads, self.dn, self.dr, self.kv_rank
+        q = q2[:, :H * (dn + dr)].unflatten(1, (H, dn + dr))
         torch.bmm(q[:, :, :dn].transpose(0, 1), self.w_uk, out=qa[:, :, :R].transpose(0, 1))
-        if dr > 0:
-            K.rotate_pairs(q2, dn, dn + dr, qa.view(T, -1), R, self.row, H, dr, rot_dims, cos_sin, pairing=self.pairing)
-        o = torch.empty(T, H, R, dtype=h.dtype, device=h.device)
-        if h.dtype == torch.bfloat16 and K.latent_attention_fits(R, dr) and latent.stride(0) % 8 == 0:
-            K.latent_prompt_attention(qa.view(T, -1), latent, H, R, dr, self.scale, self.window, batch, self.page_size, o.view(T, -1))
+        o = torch.empty(T, H, R, dtype=qa.dtype, device=qa.device)
+        if qa.dtype == torch.bfloat16 and K.latent_attention_fits(R, dr) and latent.stride(0) % 8 == 0:
+            some = {} if plan is None else {"portions": plan.rest_portions, "n_portions": len(plan.rest), "longest": plan.rest_longest}
+            K.latent_prompt_attention(qa.view(T, -1), latent, H, R, dr, self.scale, self.window, batch, self.page_size, o.view(T, -1), **some)
         else:
             K.latent_attention(qa.view(T, -1), latent, H, R, dr, self.scale, self.window, batch, self.page_size, o.view(T, -1))
-        out = torch.empty(T, H, self.dv, dtype=h.dtype, device=h.device)
-        torch.bmm(o.transpose(0, 1), self.w_uv_t, out=out.transpose(0, 1))
+        torch.bmm(o.transpose(0, 1), self.w_uv_t, out=out.view(T, H, self.dv).transpose(0, 1))
         if self.gate_act is not None:
-            gate_col = q_cols + (0 if self.shares else R + dr)
-            K.gate_cols(out.view(T, H * self.dv), y, gate_col, H * self.dv, self.gate_group, self.gate_act)
-        return linear(out.view(T, H * self.dv), self.w_o)
+            K.gate_cols(out, y, self.gate_col, H * self.dv, self.gate_group, self.gate_act)
 
 
 class TiedGateMixer:

@@ -86,7 +86,8 @@ class LatentPrepareArgs(ctypes.Structure):
                 ("kv_col", ctypes.c_int), ("kv_rank", ctypes.c_int), ("rot_dim", ctypes.c_int), ("rot_dims", ctypes.c_int),
                 ("kv_norm_w", ctypes.c_void_p), ("cos_sin", ctypes.c_void_p), ("eps", ctypes.c_float), ("cache", ctypes.c_void_p),
                 ("cache_row", ctypes.c_int64), ("slot_of_tok", ctypes.c_void_p), ("n_tok", ctypes.c_int), ("kv_out", ctypes.c_void_p),
-                ("kv_out_ld", ctypes.c_int64), ("pairing", ctypes.c_int)]
+                ("kv_out_ld", ctypes.c_int64), ("pairing", ctypes.c_int), ("rq_heads", ctypes.c_int), ("rq_col", ctypes.c_int),
+                ("rq_head", ctypes.c_int64), ("rq_out", ctypes.c_void_p), ("rq_out_ld", ctypes.c_int64), ("rq_out_head", ctypes.c_int64)]
 
 
 class AttnPrepareArgs(ctypes.Structure):
@@ -109,6 +110,7 @@ class PagedAttentionArgs(ctypes.Structure):
                 ("out", ctypes.c_void_p), ("out_ld", ctypes.c_int64), ("out_scale", ctypes.c_float),
                 ("k_row", ctypes.c_int64), ("v_row", ctypes.c_int64), ("pool", ctypes.c_int), ("pool_base", ctypes.c_int64),
                 ("v_shared", ctypes.c_int), ("out_f32", ctypes.c_int), ("out_head", ctypes.c_int64),
+                ("gate", ctypes.c_void_p), ("gate_ld", ctypes.c_int64), ("gate_group", ctypes.c_int), ("gate_act", ctypes.c_int),
                 ("chunk", ctypes.c_int)]
 
 
@@ -118,7 +120,26 @@ class PromptAttentionArgs(ctypes.Structure):
                 ("longest", ctypes.c_int), ("pages", ctypes.c_void_p), ("pages_ld", ctypes.c_int), ("page_size", ctypes.c_int),
                 ("heads", ctypes.c_int), ("kv_heads", ctypes.c_int), ("d", ctypes.c_int), ("scale", ctypes.c_float), ("window", ctypes.c_int),
                 ("keep_first", ctypes.c_int), ("sink", ctypes.c_void_p), ("pool", ctypes.c_int), ("pool_base", ctypes.c_int64),
-                ("every_value_head", ctypes.c_int), ("chunk", ctypes.c_int)]
+                ("every_value_head", ctypes.c_int), ("chunk", ctypes.c_int), ("gate", ctypes.c_void_p), ("gate_ld", ctypes.c_int64),
+                ("gate_group", ctypes.c_int), ("gate_act", ctypes.c_int)]
+
+
+class PromptAttentionTcArgs(ctypes.Structure):
+    _fields_ = [("q", ctypes.c_void_p), ("k", ctypes.c_void_p), ("k_shared", ctypes.c_void_p), ("v", ctypes.c_void_p),
+                ("q_ld", ctypes.c_int64), ("k_ld", ctypes.c_int64), ("k_shared_ld", ctypes.c_int64), ("v_ld", ctypes.c_int64),
+                ("q_rows", ctypes.c_int64), ("k_rows", ctypes.c_int64), ("out", ctypes.c_void_p), ("out_ld", ctypes.c_int64),
+                ("segments", ctypes.c_void_p), ("n_segments", ctypes.c_int), ("longest", ctypes.c_int), ("heads", ctypes.c_int),
+                ("kv_heads", ctypes.c_int), ("dn", ctypes.c_int), ("dr", ctypes.c_int), ("dv", ctypes.c_int), ("scale", ctypes.c_float),
+                ("gate", ctypes.c_void_p), ("gate_ld", ctypes.c_int64), ("gate_group", ctypes.c_int), ("gate_act", ctypes.c_int)]
+
+
+class LatentAttentionArgs(ctypes.Structure):
+    _fields_ = [("q", ctypes.c_void_p), ("q_ld", ctypes.c_int64), ("cache", ctypes.c_void_p), ("cache_row", ctypes.c_int64),
+                ("out", ctypes.c_void_p), ("out_ld", ctypes.c_int64), ("portions", ctypes.c_void_p), ("cu_tok", ctypes.c_void_p),
+                ("past", ctypes.c_void_p), ("n_portions", ctypes.c_int), ("longest", ctypes.c_int), ("pages", ctypes.c_void_p),
+                ("pages_ld", ctypes.c_int), ("page_size", ctypes.c_int), ("heads", ctypes.c_int), ("kv_rank", ctypes.c_int),
+                ("rot_dim", ctypes.c_int), ("scale", ctypes.c_float), ("window", ctypes.c_int), ("splits", ctypes.c_int),
+                ("scratch", ctypes.c_void_p)]
 
 
 SCAN_SEGMENT = 256                  # tokens per segment when a long portion is scanned as segments side by side
@@ -423,15 +444,18 @@ def attention_prepare(y, q_col, k_col, v_col, norm_mode, q_norm_w, k_norm_w, eps
 
 def paged_attention(y, q_col, k_cache, v_cache, heads, kv_heads, dk, dv, scale, window, keep_first, sink, batch, page_size, out, out_col=0,
                     out_scale=1.0, tok_index=None, k_row=0, v_row=0, pool=0, pool_base=0, v_shared=False, v_col=0, out_head=0,
-                    chunk=0):
+                    chunk=0, gate=None, gate_col=0, gate_group=1, gate_act=ACT_NONE):
     """Every token of the step (or those listed in tok_index) against the pages of its sequence: position i sees j <= i
     with i - j < window (0: all) or j < keep_first; sink [heads] f32 or None.  k_row / v_row: elements between the cache
     rows of neighbouring slots (0: kv_heads * dk / kv_heads * dv).  pool > 0: besides the window, one averaged entry per
     block of `pool` positions wholly before it, read from cache rows pool_base.. (`pool_blocks`).  v_shared: every head
     reads value columns [v_col, v_col + dv) of a row — dv is then several (or all) value heads side by side, and out_head the
     distance between the heads of an output row.  An f32 `out` is written as f32 whatever the activation type.
-    chunk > 0: a position sees only its own chunk of `chunk` positions, counted from position 0."""
+    chunk > 0: a position sees only its own chunk of `chunk` positions, counted from position 0.  gate: the result is multiplied by
+    gate_act of gate's columns from gate_col, one per `gate_group` neighbouring entries (1 or dv)."""
     a = PagedAttentionArgs()
+    if gate is not None:
+        a.gate, a.gate_ld, a.gate_group, a.gate_act = _p(gate, gate_col).value, gate.stride(0), gate_group, gate_act
     a.k_row, a.v_row = int(k_row), int(v_row)
     a.pool, a.pool_base, a.v_shared = int(pool), int(pool_base), int(bool(v_shared))
     a.out_f32 = int(out.dtype == torch.float32 and y.dtype != torch.float32)
@@ -446,23 +470,42 @@ def paged_attention(y, q_col, k_cache, v_cache, heads, kv_heads, dk, dv, scale, 
     _ok(lib().mrs_seq_paged_attention(ctypes.byref(a), _st(y)), "paged_attention")
 
 
-def dense_prompt_attention(q, q_col, k, v, batch, heads, kv_heads, d, scale, window, sink, out, out_col=0):
-    """The tensor-core prompt kernel over keys and values that are DENSE rows of the step (k, v [T, kv_heads * d], row t = the
-    step's token t) instead of pages: for steps whose sequences all start in this step with a long portion.  The kernel's page
-    table becomes one row per sequence listing its tokens' rows (page size 1); built once per step."""
-    if len(batch.long) != batch.n_seq or any(past for _, _, past, _ in batch.long):
-        raise ValueError("dense keys cover the step's own tokens only: every sequence must start in this step with a long portion")
-    plan = batch.__dict__.get("_dense_rows")
-    if plan is None:
-        rows = batch.long_rows.view(-1, 4)
-        table = (rows[:, 0:1] + torch.arange(batch.longest, dtype=torch.int32, device=rows.device)[None, :]).contiguous()
-        portions = rows.clone()
-        portions[:, 3] = torch.arange(rows.shape[0], dtype=torch.int32, device=rows.device)
-        plan = batch.__dict__["_dense_rows"] = (table, portions.contiguous())
-    table, portions = plan
-    _ok(lib().mrs_seq_prompt_attention_pooled(_p(q, q_col), _l(q.stride(0)), _p(k), _p(v), _p(out, out_col), _l(out.stride(0)), _p(portions),
-                                              _i(len(batch.long)), _i(batch.longest), _p(table), _i(table.shape[1]), _i(1), _i(heads), _i(kv_heads),
-                                              _i(d), _f(scale), _i(int(window)), _i(0), _p(sink), _i(0), _l(0), _i(0), _st(q)), "dense_prompt_attention")
+def tc_attention_fits(dn, dr, dv, *multiples_of_8):
+    """True when `tc_attention` takes these head sizes (bf16) and every given stride / first column keeps rows 16-byte aligned."""
+    return all(int(v) % 8 == 0 for v in multiples_of_8) and bool(lib().mrs_seq_prompt_attention_tc_fits(_i(dn), _i(dr), _i(dv)))
+
+
+def tc_attention(q, q_col, k, k_col, v, v_col, segments, n_segments, longest, heads, kv_heads, dn, dr, dv, scale, out, out_col=0, k_shared=None,
+                 k_shared_col=0, gate=None, gate_col=0, gate_group=1, gate_act=ACT_NONE):
+    """Causal attention of segments over DENSE keys and values on tcgen05 (bf16): segments int32 [n, 4] on the device = first query
+    row, query rows, first key row, keys before the first query.  q rows: heads * (dn + dr) columns from q_col; k: kv_heads * dn;
+    v: kv_heads * dv; k_shared: dr further key columns all heads share.  gate: as for `paged_attention`."""
+    a = PromptAttentionTcArgs()
+    a.q, a.k, a.v, a.q_ld, a.k_ld, a.v_ld = _p(q, q_col).value, _p(k, k_col).value, _p(v, v_col).value, q.stride(0), k.stride(0), v.stride(0)
+    a.q_rows, a.k_rows = q.shape[0], k.shape[0]
+    if dr > 0:
+        a.k_shared, a.k_shared_ld = _p(k_shared, k_shared_col).value, k_shared.stride(0)
+    a.out, a.out_ld = _p(out, out_col).value, out.stride(0)
+    a.segments, a.n_segments, a.longest = segments.data_ptr(), int(n_segments), int(longest)
+    a.heads, a.kv_heads, a.dn, a.dr, a.dv, a.scale = heads, kv_heads, dn, dr, dv, float(scale)
+    if gate is not None:
+        a.gate, a.gate_ld, a.gate_group, a.gate_act = _p(gate, gate_col).value, gate.stride(0), gate_group, gate_act
+    _ok(lib().mrs_seq_prompt_attention_tc(ctypes.byref(a), _st(q)), "prompt_attention_tc")
+
+
+def tc_attention_timeouts():
+    """Non-zero when a wait inside `tc_attention`'s kernel ever ran out (synchronises)."""
+    return int(lib().mrs_seq_prompt_attention_tc_timeouts())
+
+
+def gather_rows(cache, cols, runs, n_runs, longest, batch, page_size, n_rows):
+    """Dense rows [n_rows, cols] of a token-indexed cache [slots, >= cols]: runs int32 [n, 4] on the device = sequence, first
+    position, positions, first dense row.  Rows are whole 16-byte groups."""
+    out = torch.empty(n_rows, cols, dtype=cache.dtype, device=cache.device)
+    size = cache.element_size()
+    _ok(lib().mrs_seq_gather_rows(_p(cache), _l(cache.stride(0) * size), _i(cols * size), _p(runs), _i(n_runs), _i(longest), _p(batch.pages),
+                                  _i(batch.pages.shape[1]), _i(page_size), _p(out), _l(cols * size), _st(cache)), "gather_rows")
+    return out
 
 
 def pool_rows(n_token_slots, page_size, pool):
@@ -491,12 +534,14 @@ def gate_cols(x, gate, gate_col, cols, group, act):
 
 
 def prompt_attention(y, q_col, k_cache, v_cache, batch, page_size, heads, kv_heads, d, scale, window, keep_first, sink, out, out_col=0, pool=0,
-                     pool_base=0, every_value_head=False, chunk=0):
+                     pool_base=0, every_value_head=False, chunk=0, gate=None, gate_col=0, gate_group=1, gate_act=ACT_NONE):
     """The long portions of the step (batch.long: fresh or continued) on tensor cores: queries from their rows of y, keys
     and values from the pages (bf16, head size 64 or 128).  pool / pool_base: averaged blocks before the window, as for
     `paged_attention`.  every_value_head: `out` is f32 [T, heads * kv_heads * d], every head's weights on every value head.
-    chunk > 0: a position sees only its own chunk of `chunk` positions, counted from position 0."""
+    chunk > 0: a position sees only its own chunk of `chunk` positions, counted from position 0.  gate: as for `paged_attention`."""
     a = PromptAttentionArgs()
+    if gate is not None:
+        a.gate, a.gate_ld, a.gate_group, a.gate_act = _p(gate, gate_col).value, gate.stride(0), gate_group, gate_act
     a.q, a.q_ld, a.k_cache, a.v_cache = _p(y, q_col).value, y.stride(0), k_cache.data_ptr(), v_cache.data_ptr()
     a.out, a.out_ld = _p(out, out_col).value, out.stride(0)
     a.portions, a.n_portions, a.longest = batch.long_rows.data_ptr(), len(batch.long), max(n for _, n, _, _ in batch.long)
@@ -605,9 +650,11 @@ def soft_cap(x, scale, cap):
 
 # ---- attention through a shared latent -----------------------------------------------------------------------
 def latent_prepare(y, q_col, q_rank, q_norm_w, q_out, kv_col, kv_rank, rot_dim, rot_dims, kv_norm_w, cos_sin, eps, cache, slot_of_tok, kv_out=None,
-                   pairing=PAIRS_NEIGHBOURS):
+                   pairing=PAIRS_NEIGHBOURS, rotate_q=None):
     """From the columns of y: q_out = rms_norm(query latent) * w; cache[slot] = rms_norm(key/value latent) * w | the shared key
-    part turned in pairs (`pairing`).  kv_rank 0: only the query part.  kv_out [T, >= kv_rank]: the normed latent also as dense rows."""
+    part turned in pairs (`pairing`).  kv_rank 0: only the query part.  kv_out [T, >= kv_rank]: the normed latent (and, with
+    room for it, the shared key part) also as dense rows.  rotate_q = (heads, first column in y, columns between heads, out, first
+    column in out, columns between heads in out): the queries' rotated parts [rot_dim] turn in the same pass (out may be y)."""
     a = LatentPrepareArgs()
     a.y, a.y_ld, a.dtype = _p(y).value, y.stride(0), DTYPE_CODE[y.dtype]
     a.q_col, a.q_rank, a.q_norm_w = int(q_col), int(q_rank), _p(q_norm_w).value
@@ -620,6 +667,10 @@ def latent_prepare(y, q_col, q_rank, q_norm_w, q_out, kv_col, kv_rank, rot_dim, 
     a.n_tok, a.pairing = y.shape[0], pairing
     if kv_out is not None:
         a.kv_out, a.kv_out_ld = _p(kv_out).value, kv_out.stride(0)
+    if rotate_q is not None:
+        heads, col, step, dst, dst_col, dst_step = rotate_q
+        a.rq_heads, a.rq_col, a.rq_head = int(heads), int(col), int(step)
+        a.rq_out, a.rq_out_ld, a.rq_out_head = _p(dst, dst_col).value, dst.stride(0), int(dst_step)
     _ok(lib().mrs_seq_latent_prepare(ctypes.byref(a), _st(y)), "latent_prepare")
 
 
@@ -637,13 +688,27 @@ def latent_attention_fits(kv_rank, rot_dim):
     return bool(lib().mrs_seq_latent_attention_fits(_i(kv_rank), _i(rot_dim)))
 
 
-def latent_prompt_attention(qa, latent, heads, kv_rank, rot_dim, scale, window, batch, page_size, out):
-    """Absorbed latent attention of every sequence of the step on tensor cores: prompt portions of any length and single
-    decoded tokens alike (a token's heads are rows of one tile; the window's latents are fetched once for all of them)."""
-    _ok(lib().mrs_seq_latent_attention(_p(qa), _l(qa.stride(0)), _p(latent), _l(latent.stride(0)), _p(out), _l(out.stride(0)),
-                                       _p(None), _p(batch.cu_tok), _p(batch.past), _i(batch.n_seq), _i(batch.longest), _p(batch.pages),
-                                       _i(batch.pages.shape[1]), _i(page_size), _i(heads), _i(kv_rank), _i(rot_dim), _f(scale), _i(int(window)),
-                                       _st(qa)), "latent_attention")
+def latent_prompt_attention(qa, latent, heads, kv_rank, rot_dim, scale, window, batch, page_size, out, portions=None, n_portions=0, longest=0):
+    """Absorbed latent attention on tensor cores of every sequence of the step — prompt portions of any length and single
+    decoded tokens alike (a token's heads are rows of one tile; the window's latents are fetched once for all of them) — or of
+    the given portions int32 [n, 4] on the device (first row of qa / out, rows, positions cached before, sequence).  Steps too
+    small to fill the GPU share a row tile's keys among several CTAs."""
+    a = LatentAttentionArgs()
+    a.q, a.q_ld, a.cache, a.cache_row, a.out, a.out_ld = _p(qa).value, qa.stride(0), _p(latent).value, latent.stride(0), _p(out).value, out.stride(0)
+    if portions is None:
+        a.cu_tok, a.past, a.n_portions, a.longest = batch.cu_tok.data_ptr(), batch.past.data_ptr(), batch.n_seq, batch.longest
+    else:
+        a.portions, a.n_portions, a.longest = portions.data_ptr(), int(n_portions), int(longest)
+    a.pages, a.pages_ld, a.page_size = batch.pages.data_ptr(), batch.pages.shape[1], page_size
+    a.heads, a.kv_rank, a.rot_dim, a.scale, a.window = heads, kv_rank, rot_dim, float(scale), int(window)
+    reach = batch.pages.shape[1] * page_size                     # the same for every replay of a captured step
+    floats = ctypes.c_int64(0)
+    a.splits = lib().mrs_seq_latent_attention_plan(_i(a.n_portions), _i(a.longest), _i(heads), _i(kv_rank),
+                                                   _i(min(reach, window) if window > 0 else reach), ctypes.byref(floats))
+    if a.splits > 1:
+        scratch = torch.empty(floats.value, dtype=torch.float32, device=qa.device)
+        a.scratch = scratch.data_ptr()
+    _ok(lib().mrs_seq_latent_attention_general(ctypes.byref(a), _st(qa)), "latent_attention")
 
 
 def latent_attention(qa, latent, heads, kv_rank, rot_dim, scale, window, batch, page_size, out, tok_index=None):
