@@ -1187,6 +1187,147 @@ def bench_kibotar(torch, dev, peaks, steps=3, warmup=3, widths=(2048, 4096), pro
     return out
 
 
+# ------------------------------------------------------------------------------------------- --arch pikasun
+def pikasun_bench_config(width, vocab=32000):
+    """Four layers at sizes of a real model's layers of this width: latent attention (rotated part of 64, YaRN), chunked attention,
+    latent attention on the first layer's latents, chunked attention; gated feed-forwards with the weights of a plain one of four
+    times the width."""
+    H = width // 128
+    lat = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+           "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    att = {"heads": H, "kv_heads": max(1, H // 8), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+           "rot": {"base": 1000000.0, "dims": 64}}
+    mlp = {"kind": "dense", "ff": -(-8 * width // 3) // 256 * 256, "limit": 7.0}
+    return {"architecture": "Pikasun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_scale": 0.5, "logit_softcap": 30.0,
+            "layers": [{"type": "latent_attention", "mixer": lat, "mlp": mlp}, {"type": "attention", "mixer": att, "mlp": mlp},
+                       {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": mlp}, {"type": "attention", "mixer": att, "mlp": mlp}]}
+
+
+def bench_pikasun(torch, dev, peaks, steps=3, warmup=3, widths=(2048, 4096), prompt=4096, decode_batches=(1, 32)):
+    """Prefill and decode throughput of the Pikasun design through `engine.Engine.execute` at layer sizes of a real model, and of
+    the Kibotar design (the closest model: one f32 residual, latent attention over one cached row per token, grouped-query
+    attention of limited reach with an output gate, dense feed-forwards, same engine and kernel library) at equal width / depth
+    / head sizes; then, per kernel, the achieved fraction of the measured HBM rate (or of the sustained tensor rate) beside the
+    like kernel of Kibotar.  CUDA events, L2 flushed between repetitions."""
+    import numpy as np
+    from mistralrs_b200 import kibotar, pikasun
+    hbm = peaks.get("hbm_gbs", 6650.0)
+    tpeak = peaks.get("bf16_tflops_sustained", 1400.0)
+    warmup, steps = max(3, warmup), max(1, steps)
+    names = ["embed_scaled", "embed_pair", "streams_read_norm", "rms_residual", "glu_split", "gated_group_norm", "causal_conv", "linear_scan",
+             "activate_cols", "power_gate", "latent_prepare", "rotate_pairs", "latent_prompt_attention", "paged_attention", "prompt_attention",
+             "tc_attention", "gather_rows", "attention_prepare", "rotation_table", "pool_blocks", "mix_heads", "gate_cols", "soft_cap", "scale_rows"]
+    measure = engine_bench_tools(torch, dev, steps, warmup, prompt, decode_batches, names)
+    out = {"metric": "pikasun_prefill_tok_s", "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warmup, "higher_is_better": True,
+           "dtype": "bf16 (f32 residual, norms, angles, softmax)", "data": "synthetic", "sizes": []}
+    for width in widths:
+        rng = np.random.default_rng(width)
+        cj = pikasun_bench_config(width)
+        cfg = pikasun.PikasunConfig(cj)
+        model = pikasun.PikasunModel.random(cfg, dev, torch.bfloat16, seed=width)
+        row = {"width": width, "layers": len(cj["layers"]), "prompt_tokens": prompt}
+        row.update(measure(model, cfg.vocab, rng))
+        row["tc_attention_by_kind"] = pikasun_attention_alone(torch, dev, model, rng, prompt)
+        del model
+        torch.cuda.empty_cache()
+        kcj = kibotar_bench_config(width)
+        kcfg = kibotar.KibotarConfig(kcj)
+        kmodel = kibotar.KibotarModel.random(kcfg, dev, torch.bfloat16, seed=width, decay_rank=64)
+        row["kibotar_equal_size"] = near = measure(kmodel, kcfg.vocab, rng)
+        del kmodel
+        torch.cuda.empty_cache()
+        # ---- per kernel: achieved rate on the algorithmic bytes / flops of the prefill, beside the like kernel ----
+        T, W, H, d = prompt, width, width // 128, 128
+        lat, att, ff = cj["layers"][0]["mixer"], cj["layers"][1]["mixer"], cj["layers"][0]["mlp"]["ff"]
+        R, dr, G, chunk = lat["kv_rank"], lat["rot_dim"], att["kv_heads"], att["mask"]["size"]
+        katt = kcj["layers"][1]["mixer"]
+        kG, kwin, kpool = katt["kv_heads"], katt["mask"]["size"], katt["mask"]["pool"]
+        ops, kops, kinds = row["prefill_ms_by_op"], near["prefill_ms_by_op"], row["tc_attention_by_kind"]
+        gbs = lambda nbytes, ms: nbytes / (ms * 1e-3) / 1e9 / hbm if ms else None
+        tfl = lambda flop, ms: flop / (ms * 1e-3) / 1e12 if ms else None
+        tfrac = lambda flop, ms: (tfl(flop, ms) or 0.0) / tpeak
+        roof = {}
+        res = 8 * T * W * (4 + 4 + 2 + 2) + T * W * (4 + 2)             # residual read and written (f32), y read, next input written (bf16)
+        roof["rms_residual (layer norm with bias)"] = {"ms": ops.get("rms_residual"), "hbm_frac": gbs(res, ops.get("rms_residual")), "like": "rms_residual (norm before and after)",
+                                                       "like_ms": kops.get("rms_residual"), "like_hbm_frac": gbs(res, kops.get("rms_residual"))}
+        roof["embed_scaled"] = {"ms": ops.get("embed_scaled"), "hbm_frac": gbs(T * W * (2 + 4), ops.get("embed_scaled")), "like": "embed_pair",
+                                "like_ms": kops.get("embed_pair"), "like_hbm_frac": gbs(T * W * (2 + 2 + 4), kops.get("embed_pair"))}
+        prep = T * 2 * (R + dr) * 3 + 2 * T * H * dr * 2 * 2            # one layer's latent columns read, cache and dense rows written; two layers' queries turned
+        kprep = 2 * T * 2 * R * 3
+        roof["latent_prepare (norm, cache write, turned parts)"] = {"ms": ops.get("latent_prepare"), "hbm_frac": gbs(prep, ops.get("latent_prepare")), "like": "latent_prepare",
+                                                                    "like_ms": kops.get("latent_prepare"), "like_hbm_frac": gbs(kprep, kops.get("latent_prepare"))}
+        causal = T * (T + 1) / 2
+        seen = sum(min(i + 1, kwin) + max(0, i - kwin + 1) // kpool for i in range(T))
+        klat = 2 * 2.0 * H * 2 * d * causal                              # Kibotar's two causal latent layers: dk + dv multiply-adds per (query, key, head)
+        lflop = 2.0 * H * (2 * d + dr) * causal                          # one latent layer
+        aflop = 2.0 * H * 2 * d * sum(i % chunk + 1 for i in range(T))   # one chunked layer
+        roof["tc_attention (latent, decompressed, 128 + 64 / 128, causal; one layer)"] = {
+            "ms": kinds["latent"], "tflops": tfl(lflop, kinds["latent"]), "tensor_frac": tfrac(lflop, kinds["latent"]), "like": "tc_attention (128 / 128, causal; two layers)",
+            "like_ms": kops.get("tc_attention"), "like_tflops": tfl(klat, kops.get("tc_attention")), "like_tensor_frac": tfrac(klat, kops.get("tc_attention"))}
+        roof["tc_attention (chunks of %d, 128 / 128; one layer)" % chunk] = {
+            "ms": kinds["chunked"], "tflops": tfl(aflop, kinds["chunked"]), "tensor_frac": tfrac(aflop, kinds["chunked"]), "like": "prompt_attention (window + averaged blocks, executed)",
+            "like_ms": kops.get("prompt_attention"), "like_tflops": tfl(kG * 2.0 * H * 2 * d * seen, kops.get("prompt_attention")),
+            "like_tensor_frac": tfrac(kG * 2.0 * H * 2 * d * seen, kops.get("prompt_attention"))}
+        aprep = 2 * T * (2 * H * d + 2 * G * d) * 2 + 2 * T * 2 * G * d * 2
+        kaprep = T * 2 * (2 * H * d + 2 * kG * d + 2 * kG * d) + T * 2 * kG * d * 2
+        roof["attention_prepare (whole-projection norm, neighbour pairs; two layers)"] = {
+            "ms": ops.get("attention_prepare"), "hbm_frac": gbs(aprep, ops.get("attention_prepare")), "like": "attention_prepare (no norm; one layer)",
+            "like_ms": kops.get("attention_prepare"), "like_hbm_frac": gbs(kaprep, kops.get("attention_prepare"))}
+        roof["glu_split (capped)"] = {"ms": ops.get("glu_split"), "hbm_frac": gbs(4 * T * ff * (2 * 2 + 2), ops.get("glu_split")), "like": "activate_cols",
+                                      "like_ms": kops.get("activate_cols"), "like_hbm_frac": gbs(4 * T * 4 * W * (2 + 2), kops.get("activate_cols"))}
+        roof["gather_rows (latents of the reusing layer)"] = {"ms": ops.get("gather_rows"), "hbm_frac": gbs(2 * T * (R + dr) * 2, ops.get("gather_rows"))}
+        roof["soft_cap (one row)"] = {"ms": ops.get("soft_cap")}
+        lib_ms = lambda o: o.get("linear", 0.0) + o.get("bmm", 0.0) + o.get("mm", 0.0)
+        roof["library products (linear + bmm)"] = {"ms": lib_ms(ops), "like_ms": lib_ms(kops)}
+        for bi, b in enumerate(decode_batches):
+            dk = row["decode"][bi]["ms_by_op"], near["decode"][bi]["ms_by_op"]
+            ctx = prompt // 8
+            lbytes, klbytes = 2 * b * ctx * (R + dr) * 2, 2 * b * ctx * R * 2          # two latent layers: the context's latent rows once per token
+            roof["latent_prompt_attention (decode, b=%d)" % b] = {"ms": dk[0].get("latent_prompt_attention"), "hbm_frac": gbs(lbytes, dk[0].get("latent_prompt_attention")),
+                                                                  "like": "latent_prompt_attention", "like_ms": dk[1].get("latent_prompt_attention"),
+                                                                  "like_hbm_frac": gbs(klbytes, dk[1].get("latent_prompt_attention"))}
+            abytes, kabytes = 2 * b * (ctx % chunk) * 2 * G * d * 2, b * min(ctx, kwin) * 2 * kG * d * 2
+            roof["paged_attention (decode, chunk, gate; two layers, b=%d)" % b] = {
+                "ms": dk[0].get("paged_attention"), "hbm_frac": gbs(abytes, dk[0].get("paged_attention")), "like": "paged_attention (every value head; one layer)",
+                "like_ms": dk[1].get("paged_attention"), "like_hbm_frac": gbs(kabytes, dk[1].get("paged_attention"))}
+        row["roofline"] = roof
+        out["sizes"].append(row)
+    out["value"] = out["sizes"][0]["prefill_tok_s"]
+    out["ms_per_step"] = out["sizes"][0]["prefill_ms"]
+    out["config"] = {"workload": "4 layers (latent attention 128 + 64 / 128 on a latent of 512, attention in chunks of 1024, latent attention on the first layer's "
+                                 "latents, chunked attention; gated feed-forwards of 8/3 x width), widths %s, %d-token prompt; decode at context %d; Kibotar at equal "
+                                 "sizes beside it; L2 flushed between repetitions" % (list(widths), prompt, prompt // 8)}
+    return out
+
+
+def pikasun_attention_alone(torch, dev, model, rng, prompt):
+    """ms of `tc_attention` in one latent and in one chunked layer of a whole-prompt step (events around every call, median of five
+    steps)."""
+    from mistralrs_b200 import engine, seq_ops as K
+    eng = engine.Engine(model, max_tokens=prompt + 64, max_seqs=1)
+    toks, real, calls = rng.integers(0, model.vocab, prompt).tolist(), K.tc_attention, []
+
+    def timed(*a, **k):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        real(*a, **k)
+        e1.record()
+        calls.append(("latent" if k.get("k_shared") is not None else "chunked", e0, e1))
+    K.tc_attention = timed
+    try:
+        for _ in range(8):
+            r = eng.new_request(toks)
+            eng.execute([(r, prompt)])
+            eng.finish(r)
+        torch.cuda.synchronize()
+    finally:
+        K.tc_attention = real
+    ms = {}
+    for kind, e0, e1 in calls[len(calls) * 3 // 8:]:
+        ms.setdefault(kind, []).append(e0.elapsed_time(e1))
+    return {kind: round(sorted(v)[len(v) // 2], 4) for kind, v in ms.items()}
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1196,12 +1337,13 @@ def main():
     ap.add_argument("--config", type=int, default=2, choices=[1, 2, 3, 4, 5],
                     help="headline workload: 1 = TinyLlama-1.1B Q4_K_M on the CPU (plumbing, no GPU), 2 = 8B Q4_K_M decode b=1 (default), "
                          "3 = 8B Q8_0 prefill 4096, 4 = Mistral-7B GPTQ b=32, 5 = Llama-3-70B Q4_K_M tensor parallel (needs --gpus 8)")
-    ap.add_argument("--arch", default="llama", choices=["llama", "nisasun", "kilizen", "fosulix", "kibotar"],
+    ap.add_argument("--arch", default="llama", choices=["llama", "nisasun", "kilizen", "fosulix", "kibotar", "pikasun"],
                     help="nisasun: prefill / decode throughput of the Nisasun design on the step engine at layer sizes of a real model "
                          "(random weights), beside the Llama path at equal width / depth / feed-forward size, with a per-kernel table; "
                          "kilizen: the same for the Kilizen design, beside Nisasun at equal sizes; "
                          "fosulix: the same for the Fosulix design, beside Kilizen at equal sizes; "
-                         "kibotar: the same for the Kibotar design, beside Fosulix at equal sizes")
+                         "kibotar: the same for the Kibotar design, beside Fosulix at equal sizes; "
+                         "pikasun: the same for the Pikasun design, beside Kibotar at equal sizes")
     ap.add_argument("--layers", type=int, default=0, help="debug: truncate the model")
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("MRS_PDL", "1")))
     ap.add_argument("--no-cpu-baseline", action="store_true")
@@ -1247,6 +1389,9 @@ def main():
         return
     if args.arch == "kibotar":
         print(json.dumps(bench_kibotar(torch, dev, peaks, steps=args.steps, warmup=args.warmup)))
+        return
+    if args.arch == "pikasun":
+        print(json.dumps(bench_pikasun(torch, dev, peaks, steps=args.steps, warmup=args.warmup)))
         return
     if args.config == 3 and world == 1:
         pf = bench_prefill_q8(M, torch, dev, peaks, layers=args.layers)

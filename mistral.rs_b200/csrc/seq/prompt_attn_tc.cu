@@ -6,15 +6,16 @@
 // of a chunked layer (each its own segment, nothing to mask but the diagonal), or cached rows gathered / decompressed for the
 // step.
 //
-// One CTA = 128 query rows of one (segment, head), key tiles of BN rows, 192 threads (the roles of prefill_attn_tc.cu):
-//   warp 0      TMA: Q once, then K and V tiles, in SWIZZLE_128B boxes of 64 columns;
+// One CTA = 128 query rows of one (segment, head), key tiles of 64 rows, 192 threads:
+//   warp 0      TMA: Q once, then K tiles through a 2-stage ring and V tiles, in SWIZZLE_128B boxes of 64 columns;
 //   warp 1      MMA issuer: S = Q K^T (both K-major in shared memory; 16 columns per MMA, dn / 16 + ceil(dr / 16) of them),
 //               O += P V (P in tensor memory, V from its row-major tile as an MN-major operand);
-//   warps 2..5  softmax + correction + epilogue, thread = query row = TMEM lane; P overwrites the head of S.
-// Two CTAs share an SM (one tile's softmax runs beside the other's products): BN is 128 while the tiles allow it, 64 with
-// three key boxes.  Boxes are always 64 columns wide.  Head sizes that do not fill their last box leave neighbouring columns
-// in it; the MMAs of S stop at the head's own columns (the shared part's box is filled with zeros past its end), and columns of
-// O past dv are never stored.
+//   warps 2..5  softmax + correction + epilogue, thread = query row = TMEM lane; P overwrites the head of its S.
+// S has two buffers in tensor memory: the products of tile j + 1 run beside the softmax of tile j, so the softmax warps find
+// their next scores ready; two CTAs share an SM (256 TMEM columns and at most 112 KB each).  Blocks are ordered by tile, heavy
+// (late) query tiles of all heads first.  Boxes are always 64 columns wide.  Head sizes that do not fill their last box leave
+// neighbouring columns in it; the MMAs of S stop at the head's own columns (the shared part's box is filled with zeros past its
+// end), and columns of O past dv are never stored.
 //
 // Every wait has a limit; a wait that runs out sets a device flag (mrs_seq_prompt_attention_tc_timeouts) and ends the CTA.
 #include "../tc_common.cuh"
@@ -24,7 +25,9 @@
 namespace seqtc {
 using namespace mrs;
 
-constexpr int BM = 128, THREADS = 192;
+constexpr int BM = 128, BN = 64, THREADS = 192;
+// A barrier's waiters may be at most one phase behind it, or a completed phase reads as a pending one: barriers that several
+// tiles could pass before a waiter looks (S, P and PV of two tiles are in flight at once) exist once per parity of the tile.
 constexpr uint32_t TCOLS = 256, O_COL = 128, WAIT_LIMIT = 1u << 22;
 
 struct Params {
@@ -93,10 +96,10 @@ __device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const uint32_t *r) {
 
 // NB: 64-column boxes of a head's own key columns; SH: 1 when a shared key part follows; NV: 64-column boxes of the values
 template <int NB, int SH, int NV> struct Shape {
-  static constexpr int BOXES = NB + SH, BN = BOXES > 2 ? 64 : 128;
+  static constexpr int BOXES = NB + SH;
   static constexpr int QBOX = BM * 128, KBOX = BN * 128;                      // bytes of one box
   static constexpr int Q_BYTES = BOXES * QBOX, K_BYTES = BOXES * KBOX, V_BYTES = NV * KBOX;
-  static constexpr int SMEM = 1024 + Q_BYTES + K_BYTES + V_BYTES + 256;
+  static constexpr int SMEM = Q_BYTES + 2 * K_BYTES + V_BYTES + 256;
 };
 
 template <int NB, int SH, int NV>
@@ -104,27 +107,29 @@ __global__ void __launch_bounds__(THREADS, 2)
 prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                            const __grid_constant__ CUtensorMap tmap_ks, const __grid_constant__ CUtensorMap tmap_v, const Params p) {
   using S = Shape<NB, SH, NV>;
-  constexpr int BN = S::BN;
-  extern __shared__ __align__(1024) uint8_t smem_raw[];
-  uint8_t *smem = (uint8_t *)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  uint8_t *q_s = smem, *k_s = q_s + S::Q_BYTES, *v_s = k_s + S::K_BYTES;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  uint8_t *q_s = smem, *k_s = q_s + S::Q_BYTES, *v_s = k_s + 2 * S::K_BYTES;
   uint64_t *bars = (uint64_t *)(v_s + S::V_BYTES);
-  uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 2, *v_full = bars + 3, *v_empty = bars + 4, *s_full = bars + 5,
-           *p_full = bars + 6, *pv_done = bars + 7;
-  uint32_t *tmem_slot = (uint32_t *)(bars + 8);
+  uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 3, *v_full = bars + 5, *v_empty = bars + 6, *s_full = bars + 7,
+           *p_full = bars + 9, *pv_done = bars + 11;                 // k_*, s_full, p_full, pv_done: one per parity of j
+  uint32_t *tmem_slot = (uint32_t *)(bars + 13);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h = blockIdx.y, kvh = h / (p.H / p.KVH);
+  const int h = blockIdx.x, kvh = h / (p.H / p.KVH);
   const int32_t *seg = p.segments + 4 * blockIdx.z;
   const int row0 = seg[0], len = seg[1], key0 = seg[2], past = seg[3];
-  const int qt = (len + BM - 1) / BM - 1 - (int)blockIdx.x;          // heavy (late) query tiles first
+  const int qt = (len + BM - 1) / BM - 1 - (int)blockIdx.y;          // heavy (late) query tiles first
   if (qt < 0) return;
+  if (smem_u32(smem) & 1023) {                                       // the swizzled boxes need it; never seen
+    if (tid == 0) atomicExch(&g_timeouts, 2);
+    return;
+  }
   const int q0 = qt * BM;
   const int kv_end = past + min(len, q0 + BM);
   const int nt = (kv_end + BN - 1) / BN;                             // >= 1
 
-  if (warp == 0 && lane < 8) {
-    mbar_init(&bars[lane], lane == 6 ? 4u : 1u);                     // p_full: the four softmax warps
+  if (warp == 0 && lane < 13) {
+    mbar_init(&bars[lane], lane == 9 || lane == 10 ? 4u : 1u);       // p_full: the four softmax warps
     fence_mbar_init();
   }
   if (warp == 1) tmem_alloc(tmem_slot, TCOLS);
@@ -132,33 +137,37 @@ prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = __reduce_max_sync(0xffffffffu, *tmem_slot);
-  const uint32_t t_s = tmem_base, t_p = tmem_base, t_o = tmem_base + O_COL;      // P overwrites the head of S
+  const uint32_t t_s = tmem_base, t_o = tmem_base + O_COL;           // S and P of tile j: columns t_s + BN * (j & 1) ..
 
   if (warp == 0) {
-    // ===================== TMA producer =====================
+    // ===================== TMA producer: K_0, then K_{j+1} and V_j =====================
     const int qx = h * (p.dn + p.dr);
     mbar_arrive_expect_tx_warp(q_full, S::Q_BYTES);
 #pragma unroll
     for (int i = 0; i < NB; i++) tma_load_2d_warp(q_s + i * S::QBOX, &tmap_q, qx + 64 * i, row0 + q0, q_full);
     if (SH) tma_load_2d_warp(q_s + NB * S::QBOX, &tmap_q, qx + p.dn, row0 + q0, q_full);
     int k_issued = 0, v_issued = 0;
-    for (int j = 0; j < nt; j++) {
-      const int ph = j & 1, row = key0 + j * BN;
-      if (!wait_limited(k_empty, ph ^ 1)) break;
-      mbar_arrive_expect_tx_warp(k_full, S::K_BYTES);
+    for (int j = -1; j < nt; j++) {
+      if (j + 1 < nt) {
+        const int b = (j + 1) & 1, row = key0 + (j + 1) * BN;
+        uint8_t *dst = k_s + b * S::K_BYTES;
+        if (!wait_limited(k_empty + b, (((j + 1) >> 1) & 1) ^ 1)) break;
+        mbar_arrive_expect_tx_warp(k_full + b, S::K_BYTES);
 #pragma unroll
-      for (int i = 0; i < NB; i++) tma_load_2d_warp(k_s + i * S::KBOX, &tmap_k, kvh * p.dn + 64 * i, row, k_full);
-      if (SH) tma_load_2d_warp(k_s + NB * S::KBOX, &tmap_ks, 0, row, k_full);
-      k_issued = j + 1;
-      if (!wait_limited(v_empty, ph ^ 1)) break;
+        for (int i = 0; i < NB; i++) tma_load_2d_warp(dst + i * S::KBOX, &tmap_k, kvh * p.dn + 64 * i, row, k_full + b);
+        if (SH) tma_load_2d_warp(dst + NB * S::KBOX, &tmap_ks, 0, row, k_full + b);
+        k_issued = j + 2;
+      }
+      if (j < 0) continue;
+      if (!wait_limited(v_empty, (j & 1) ^ 1)) break;
       mbar_arrive_expect_tx_warp(v_full, S::V_BYTES);
 #pragma unroll
-      for (int i = 0; i < NV; i++) tma_load_2d_warp(v_s + i * S::KBOX, &tmap_v, kvh * p.dv + 64 * i, row, v_full);
+      for (int i = 0; i < NV; i++) tma_load_2d_warp(v_s + i * S::KBOX, &tmap_v, kvh * p.dv + 64 * i, key0 + j * BN, v_full);
       v_issued = j + 1;
     }
     if (v_issued < nt) {                 // gave up: let the copies in flight land before the CTA may end
       wait_limited(q_full, 0);
-      if (k_issued > 0) wait_limited(k_full, (k_issued - 1) & 1);
+      for (int j = max(0, k_issued - 2); j < k_issued; j++) wait_limited(k_full + (j & 1), (j >> 1) & 1);
       if (v_issued > 0) wait_limited(v_full, (v_issued - 1) & 1);
     }
   } else if (warp == 1) {
@@ -167,34 +176,41 @@ prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
     const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(NV * 64 >> 3) << 17) | ((uint32_t)(BM >> 4) << 24);
     const int own_steps = p.dn >> 4, shared_steps = SH ? (p.dr + 15) >> 4 : 0;
-    bool ok = wait_limited(q_full, 0);
-    int done = 0;                        // PV products committed
-    for (int j = 0; ok && j < nt; j++) {
-      const int ph = j & 1;
-      ok = wait_limited(k_full, ph);
-      if (ok && j > 0) ok = wait_limited(pv_done, ph ^ 1);           // PV_{j-1} has read P out of the S columns S_j overwrites
-      if (!ok) break;
+    auto scores = [&](int j) {           // S_j = Q K_j^T into buffer j & 1
+      const int b = j & 1;
+      if (!wait_limited(k_full + b, (j >> 1) & 1)) return false;
       tc_fence_after();
       for (int c = 0; c < own_steps + shared_steps; c++) {
         const int box = c < own_steps ? c >> 2 : NB, step = c < own_steps ? c & 3 : c - own_steps;
         const uint64_t ad = umma_desc_sw128(q_s + box * S::QBOX) + (uint64_t)(2 * step);
-        const uint64_t bd = umma_desc_sw128(k_s + box * S::KBOX) + (uint64_t)(2 * step);
-        umma_ss_warp(t_s, ad, bd, idesc_s, c ? 1u : 0u);
+        const uint64_t bd = umma_desc_sw128(k_s + b * S::K_BYTES + box * S::KBOX) + (uint64_t)(2 * step);
+        umma_ss_warp(t_s + (uint32_t)(BN * b), ad, bd, idesc_s, c ? 1u : 0u);
       }
-      umma_commit_warp(s_full);
-      umma_commit_warp(k_empty);
-      ok = wait_limited(p_full, ph) && wait_limited(v_full, ph);
+      umma_commit_warp(s_full + b);
+      umma_commit_warp(k_empty + b);
+      return true;
+    };
+    bool ok = wait_limited(q_full, 0) && scores(0);
+    int done = 0;                        // PV products committed
+    for (int j = 0; ok && j < nt; j++) {
+      if (j + 1 < nt) {
+        if (j > 0) ok = wait_limited(pv_done + ((j - 1) & 1), ((j - 1) >> 1) & 1);      // PV_{j-1} has read P out of the buffer S_{j+1} overwrites
+        ok = ok && scores(j + 1);
+        if (!ok) break;
+      }
+      ok = wait_limited(p_full + (j & 1), (j >> 1) & 1) && wait_limited(v_full, j & 1);
       if (!ok) break;
       tc_fence_after();
-      const uint32_t vs = smem_u32(v_s);
+      const uint32_t vs = smem_u32(v_s), t_p = t_s + (uint32_t)(BN * (j & 1));
 #pragma unroll
       for (int c = 0; c < BN / 16; c++)   // 16 keys per MMA: two 8-row groups of 1024 B; the next 64 columns one box further
         umma_f16_ts_warp(t_o, t_p + (uint32_t)(8 * c), desc_sw128_ex(vs + (uint32_t)c * 2048u, S::KBOX, 1024u), idesc_o, (j | c) ? 1u : 0u);
-      umma_commit_warp(pv_done);
+      umma_commit_warp(pv_done + (j & 1));
       umma_commit_warp(v_empty);
       done = j + 1;
     }
-    if (done > 0) wait_limited(pv_done, (done - 1) & 1);             // no product is in flight when tensor memory is freed
+    // no product is in flight when tensor memory is freed (a commit covers everything issued before it)
+    if (done > 0) wait_limited(pv_done + ((done - 1) & 1), ((done - 1) >> 1) & 1);
   } else {
     // ===================== softmax / correction / epilogue: thread = query row =====================
     const int q4 = warp & 3, r = q4 * 32 + lane;
@@ -205,10 +221,10 @@ prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     float m_ref = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int j = 0; ok && j < nt; j++) {
-      const int ph = j & 1;
-      const uint32_t ts = t_s + lane_off;
+      const int b = j & 1;
+      const uint32_t ts = t_s + (uint32_t)(BN * b) + lane_off;
       const int lim = min(qpos, kv_end - 1) - j * BN;                // columns > lim are masked
-      ok = wait_limited(s_full, ph);
+      ok = wait_limited(s_full + b, (j >> 1) & 1);
       if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
       tc_fence_after();
       uint32_t v[BN];
@@ -231,7 +247,10 @@ prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       const float m_use = move ? fmaxf(m_ref, mx) : m_ref;
       const float corr = (m_use == m_ref) ? 1.f : ex2(m_ref - m_use);
       const float msub = (m_use == -INFINITY) ? 0.f : m_use;
-      if (j > 0 && __any_sync(0xffffffffu, corr != 1.f)) {           // PV_{j-1} is complete: S_j was issued after it
+      if (j > 0 && __any_sync(0xffffffffu, corr != 1.f)) {           // O is rescaled between PV_{j-1} and PV_j
+        ok = __all_sync(0xffffffffu, wait_limited(pv_done + ((j - 1) & 1), ((j - 1) >> 1) & 1));
+        if (!ok) break;
+        tc_fence_after();
 #pragma unroll 1
         for (int c0 = 0; c0 < NV * 64; c0 += 32) {
           uint32_t o[32];
@@ -253,16 +272,16 @@ prompt_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
           const __nv_bfloat162 hh = __floats2bfloat162_rn(p0, p1);
           pk[i >> 1] = *(const uint32_t *)&hh;
         }
-        tmem_st_x16(t_p + lane_off + (uint32_t)(c0 >> 1), pk);
+        tmem_st_x16(ts + (uint32_t)(c0 >> 1), pk);
       }
       l_run = l_run * corr + rs;
       m_ref = m_use;
       tmem_wait_st();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_full);
+      if (lane == 0) mbar_arrive(p_full + b);
     }
-    if (ok) ok = __all_sync(0xffffffffu, wait_limited(pv_done, (nt - 1) & 1));
+    if (ok) ok = __all_sync(0xffffffffu, wait_limited(pv_done + ((nt - 1) & 1), ((nt - 1) >> 1) & 1));
     if (ok) {                             // O / l -> global, times the output gate
       tc_fence_after();
       const float inv = (l_run > 0.f) ? 1.f / l_run : 0.f;
@@ -321,7 +340,7 @@ static int launch(const CUtensorMap &tq, const CUtensorMap &tk, const CUtensorMa
     if (e != cudaSuccess) return (int)e;
     raised = true;
   }
-  kern<<<dim3((longest + BM - 1) / BM, p.H, n), THREADS, bytes, st>>>(tq, tk, ts, tv, p);
+  kern<<<dim3(p.H, (longest + BM - 1) / BM, n), THREADS, bytes, st>>>(tq, tk, ts, tv, p);
   return (int)cudaGetLastError();
 }
 
@@ -354,7 +373,7 @@ extern "C" int mrs_seq_prompt_attention_tc(const mrs_seq_prompt_attention_tc_arg
   using namespace seqtc;
   const mrs_seq_prompt_attention_tc_args &a = *args;
   if (a.n_segments <= 0 || a.longest <= 0) return 0;
-  if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.heads > 65535 || a.n_segments > 65535 || !a.segments || a.q_rows <= 0 || a.k_rows <= 0)
+  if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || (a.longest + BM - 1) / BM > 65535 || a.n_segments > 65535 || !a.segments || a.q_rows <= 0 || a.k_rows <= 0)
     return -2;
   if (!mrs_seq_prompt_attention_tc_fits(a.dn, a.dr, a.dv) || a.scale <= 0.0f || (a.dr > 0 && !a.k_shared)) return -2;
   if (a.gate && a.gate_group != 1 && a.gate_group != a.dv) return -2;
@@ -364,7 +383,7 @@ extern "C" int mrs_seq_prompt_attention_tc(const mrs_seq_prompt_attention_tc_arg
   if (a.gate && a.gate_group == 1 && (a.gate_ld % 8 || !al(a.gate))) return -3;
   PFN_encodeTiled enc = tc_get_encode();
   if (!enc) return -4;
-  const int nb = (a.dn + 63) / 64, sh = a.dr > 0 ? 1 : 0, nv = (a.dv + 63) / 64, bn = nb + sh > 2 ? 64 : 128;
+  const int nb = (a.dn + 63) / 64, sh = a.dr > 0 ? 1 : 0, nv = (a.dv + 63) / 64;
   auto make = [&](CUtensorMap *m, const void *base, int64_t cols, int64_t rows, int64_t ld, int box_rows) -> bool {
     const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
     const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
@@ -374,11 +393,11 @@ extern "C" int mrs_seq_prompt_attention_tc(const mrs_seq_prompt_attention_tc_arg
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
   };
   CUtensorMap tq, tk, ts, tv;
-  if (!make(&tq, a.q, (int64_t)a.heads * (a.dn + a.dr), a.q_rows, a.q_ld, BM) || !make(&tk, a.k, (int64_t)a.kv_heads * a.dn, a.k_rows, a.k_ld, bn) ||
-      !make(&tv, a.v, (int64_t)a.kv_heads * a.dv, a.k_rows, a.v_ld, bn))
+  if (!make(&tq, a.q, (int64_t)a.heads * (a.dn + a.dr), a.q_rows, a.q_ld, BM) || !make(&tk, a.k, (int64_t)a.kv_heads * a.dn, a.k_rows, a.k_ld, BN) ||
+      !make(&tv, a.v, (int64_t)a.kv_heads * a.dv, a.k_rows, a.v_ld, BN))
     return -4;
   ts = tk;
-  if (sh && !make(&ts, a.k_shared, a.dr, a.k_rows, a.k_shared_ld, bn)) return -4;
+  if (sh && !make(&ts, a.k_shared, a.dr, a.k_rows, a.k_shared_ld, BN)) return -4;
   Params p = {};
   p.o = (__nv_bfloat16 *)a.out; p.o_ld = a.out_ld; p.segments = a.segments;
   p.H = a.heads; p.KVH = a.kv_heads; p.dn = a.dn; p.dr = a.dr; p.dv = a.dv;

@@ -99,6 +99,9 @@ template <typename T> __device__ __forceinline__ float2 load2(const T *p);
 template <> __device__ __forceinline__ float2 load2<float>(const float *p) { return *(const float2 *)p; }
 template <> __device__ __forceinline__ float2 load2<__nv_bfloat16>(const __nv_bfloat16 *p) { return __bfloat1622float2(*(const __nv_bfloat162 *)p); }
 
+template <typename T> __device__ __forceinline__ void store2(T *p, float2 v);
+template <> __device__ __forceinline__ void store2<float>(float *p, float2 v) { *(float2 *)p = v; }
+template <> __device__ __forceinline__ void store2<__nv_bfloat16>(__nv_bfloat16 *p, float2 v) { *(__nv_bfloat162 *)p = __floats2bfloat162_rn(v.x, v.y); }
 
 // four neighbouring elements (the pointer is 4-element aligned)
 template <typename T> __device__ __forceinline__ float4 load4(const T *p);

@@ -84,6 +84,184 @@ __global__ void attention_prepare_kernel(const mrs_seq_attn_prepare_args a) {
   }
 }
 
+// The same with two neighbouring entries per lane and step (even head sizes, rows aligned to two entries; a halves rotation over
+// an even number of pairs): a neighbour pair is one access, halves are two pairs side by side.
+template <typename T>
+__global__ void attention_prepare_vec_kernel(const mrs_seq_attn_prepare_args a) {
+  extern __shared__ float ss[];   // [heads + kv_heads] sums of squares
+  const int t = blockIdx.x, lane = threadIdx.x & 31, wib = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int heads = a.heads, kv_heads = a.kv_heads, dk = a.dk, dv = a.dv;
+  T *q = (T *)a.q + (int64_t)t * a.q_ld, *k = (T *)a.k + (int64_t)t * a.k_ld;
+  const int64_t slot = a.slot_of_tok[t];
+  const bool normed = a.norm_mode != MRS_SEQ_QK_NORM_NONE;
+  if (normed) {
+    for (int job = wib; job < heads + kv_heads; job += nw) {
+      const T *src = job < heads ? q + job * dk : k + (job - heads) * dk;
+      float s = 0.0f;
+      for (int d = 2 * lane; d < dk; d += 64) {
+        const float2 x = load2<T>(src + d);
+        s = fmaf(x.x, x.x, fmaf(x.y, x.y, s));
+      }
+      s = warp_sum(s);
+      if (lane == 0) ss[job] = s;
+    }
+    __syncthreads();
+  }
+  float inv_q_all = 1.0f, inv_k_all = 1.0f;
+  if (a.norm_mode == MRS_SEQ_QK_NORM_WHOLE) {      // every warp sums the heads' sums across its lanes
+    float sq = 0.0f, sk = 0.0f;
+    for (int h = lane; h < heads + kv_heads; h += 32) {
+      if (h < heads) sq += ss[h];
+      else sk += ss[h];
+    }
+    inv_q_all = rsqrtf_exact(warp_sum(sq) / (float)(heads * dk) + a.eps);
+    inv_k_all = rsqrtf_exact(warp_sum(sk) / (float)(kv_heads * dk) + a.eps);
+  }
+  const int half = a.cos_sin ? a.rot_dims / 2 : 0;
+  const float2 *cs = (const float2 *)a.cos_sin + (int64_t)t * half;
+  const bool neighbours = a.pairing == MRS_SEQ_PAIRS_NEIGHBOURS;
+  for (int job = wib; job < heads + 2 * kv_heads; job += nw) {
+    if (job < heads + kv_heads) {
+      const bool is_q = job < heads;
+      const int hh = is_q ? job : job - heads;
+      T *src = is_q ? q + hh * dk : k + hh * dk;
+      const float *w = is_q ? a.q_norm_w : a.k_norm_w;
+      float inv = 1.0f;
+      if (a.norm_mode == MRS_SEQ_QK_NORM_HEAD) inv = rsqrtf_exact(ss[job] / (float)dk + a.eps);
+      else if (a.norm_mode == MRS_SEQ_QK_NORM_WHOLE) { inv = is_q ? inv_q_all : inv_k_all; w += hh * dk; }
+      T *cached = (!is_q && slot >= 0) ? (T *)a.k_cache + (slot * kv_heads + hh) * dk : nullptr;
+      if (!is_q && a.v == nullptr) {      // the values are the keys as projected
+        if (slot >= 0) {
+          T *vc = (T *)a.v_cache + (slot * kv_heads + hh) * dv;
+          for (int d = 2 * lane; d < dk; d += 64) store2<T>(vc + d, load2<T>(src + d));
+        }
+        __syncwarp();
+      }
+      auto value = [&](int d) {
+        float2 x = load2<T>(src + d);
+        if (normed) { x.x *= inv * w[d]; x.y *= inv * w[d + 1]; }
+        return x;
+      };
+      auto put = [&](int d, float2 x) {
+        store2<T>(src + d, x);
+        if (cached) store2<T>(cached + d, x);
+      };
+      if (neighbours) {
+        for (int i = lane; i < half; i += 32) {
+          const float2 x = value(2 * i), c = cs[i];
+          put(2 * i, make_float2(x.x * c.x - x.y * c.y, x.y * c.x + x.x * c.y));
+        }
+      } else {
+        for (int i = 2 * lane; i < half; i += 64) {
+          const float2 u = value(i), v = value(i + half), c0 = cs[i], c1 = cs[i + 1];
+          put(i, make_float2(u.x * c0.x - v.x * c0.y, u.y * c1.x - v.y * c1.y));
+          put(i + half, make_float2(v.x * c0.x + u.x * c0.y, v.y * c1.x + u.y * c1.y));
+        }
+      }
+      for (int d = 2 * half + 2 * lane; d < dk; d += 64) put(d, value(d));       // the rest passes
+    } else if (slot >= 0 && a.v != nullptr) {
+      const int hh = job - heads - kv_heads;
+      const T *src = (const T *)a.v + (int64_t)t * a.v_ld + hh * dv;
+      T *dst = (T *)a.v_cache + (slot * kv_heads + hh) * dv;
+      for (int d = 2 * lane; d < dv; d += 64) store2<T>(dst + d, load2<T>(src + d));
+    }
+  }
+}
+
+// The same for layers whose norm is over the whole projection (or that have none) and whose rotation is in neighbouring pairs (or
+// absent): a token's q | k entries are one flat row, eight neighbours per thread and step (16-byte accesses in bf16), one
+// reduction of two sums for the block.  Needs head sizes in whole groups of eight.
+template <typename T> __device__ __forceinline__ void load8(const T *p, float *v) {
+  const float4 a = load4<T>(p), b = load4<T>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16 *p, float *v) {
+  const uint4 raw = *(const uint4 *)p;
+  const __nv_bfloat162 *h = (const __nv_bfloat162 *)&raw;
+#pragma unroll
+  for (int i = 0; i < 4; i++) {
+    const float2 x = __bfloat1622float2(h[i]);
+    v[2 * i] = x.x;
+    v[2 * i + 1] = x.y;
+  }
+}
+template <typename T> __device__ __forceinline__ void store8(T *p, const float *v) {
+  store4<T>(p, make_float4(v[0], v[1], v[2], v[3]));
+  store4<T>(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+template <> __device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16 *p, const float *v) {
+  uint4 raw;
+  __nv_bfloat162 *h = (__nv_bfloat162 *)&raw;
+#pragma unroll
+  for (int i = 0; i < 4; i++) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+  *(uint4 *)p = raw;
+}
+
+template <typename T>
+__global__ void attention_prepare_row_kernel(const mrs_seq_attn_prepare_args a) {
+  __shared__ float red[2][32];
+  const int t = blockIdx.x, lane = threadIdx.x & 31, wib = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int dk = a.dk, qn = a.heads * dk / 8, kn = a.kv_heads * dk / 8, vn = a.v ? a.kv_heads * a.dv / 8 : 0;
+  T *q = (T *)a.q + (int64_t)t * a.q_ld, *k = (T *)a.k + (int64_t)t * a.k_ld;
+  const int64_t slot = a.slot_of_tok[t];
+  const bool normed = a.norm_mode == MRS_SEQ_QK_NORM_WHOLE;
+  float inv_q = 1.0f, inv_k = 1.0f, v[8];
+  if (normed) {
+    float sq = 0.0f, sk = 0.0f;
+    for (int e = threadIdx.x; e < qn + kn; e += blockDim.x) {
+      load8<T>(e < qn ? q + 8 * e : k + 8 * (e - qn), v);
+      float s = 0.0f;
+#pragma unroll
+      for (int i = 0; i < 8; i++) s = fmaf(v[i], v[i], s);
+      if (e < qn) sq += s;
+      else sk += s;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { red[0][wib] = sq; red[1][wib] = sk; }
+    __syncthreads();
+    sq = warp_sum(lane < nw ? red[0][lane] : 0.0f);
+    sk = warp_sum(lane < nw ? red[1][lane] : 0.0f);
+    inv_q = rsqrtf_exact(sq / (float)(8 * qn) + a.eps);
+    inv_k = rsqrtf_exact(sk / (float)(8 * kn) + a.eps);
+  }
+  const int half = a.cos_sin ? a.rot_dims / 2 : 0;
+  const float2 *cs = (const float2 *)a.cos_sin + (int64_t)t * half;
+  for (int e = threadIdx.x; e < qn + kn + vn; e += blockDim.x) {
+    if (e >= qn + kn) {
+      const int c = 8 * (e - qn - kn);
+      if (slot >= 0) {
+        load8<T>((const T *)a.v + (int64_t)t * a.v_ld + c, v);
+        store8<T>((T *)a.v_cache + slot * (8 * vn) + c, v);
+      }
+      continue;
+    }
+    const bool is_q = e < qn;
+    const int c = 8 * (is_q ? e : e - qn);
+    T *src = (is_q ? q : k) + c;
+    load8<T>(src, v);
+    if (!is_q && a.v == nullptr && slot >= 0) store8<T>((T *)a.v_cache + slot * (8 * kn) + c, v);      // the values are the keys as projected
+    if (normed) {
+      const float *w = (is_q ? a.q_norm_w : a.k_norm_w) + c, inv = is_q ? inv_q : inv_k;
+      const float4 w0 = *(const float4 *)w, w1 = *(const float4 *)(w + 4);
+      v[0] *= inv * w0.x; v[1] *= inv * w0.y; v[2] *= inv * w0.z; v[3] *= inv * w0.w;
+      v[4] *= inv * w1.x; v[5] *= inv * w1.y; v[6] *= inv * w1.z; v[7] *= inv * w1.w;
+    }
+    const int pair0 = (c % dk) / 2;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      if (pair0 + i < half) {
+        const float2 r = cs[pair0 + i];
+        const float x = v[2 * i], y = v[2 * i + 1];
+        v[2 * i] = x * r.x - y * r.y;
+        v[2 * i + 1] = y * r.x + x * r.y;
+      }
+    }
+    store8<T>(src, v);
+    if (!is_q && slot >= 0) store8<T>((T *)a.k_cache + slot * (8 * kn) + c, v);
+  }
+}
+
 // cos_sin[t][i] = mag * (cos, sin)(pos[t] * freq[i]): the angle, and its reduction, in double — positions in the thousands
 // times a frequency near one leave no digits to spare in f32
 __global__ void rotation_table_kernel(const int32_t *__restrict__ pos_of_tok, const double *__restrict__ freq, int n_tok, int half,
@@ -317,6 +495,23 @@ extern "C" int mrs_seq_attention_prepare(const mrs_seq_attn_prepare_args *args, 
   if (a.cos_sin && (a.rot_dims < 2 || a.rot_dims % 2 || a.rot_dims > a.dk)) return -2;
   const int jobs = a.heads + 2 * a.kv_heads, warps = jobs < 8 ? jobs : 8;
   const size_t bytes = (size_t)(a.heads + a.kv_heads) * sizeof(float);
+  const int two = a.dtype == MRS_SEQ_BF16 ? 4 : 8, half = a.cos_sin ? a.rot_dims / 2 : 0;
+  auto al = [two](const void *p) { return (uintptr_t)p % two == 0; };
+  auto al16 = [](const void *p) { return (uintptr_t)p % 16 == 0; };
+  if (a.norm_mode != MRS_SEQ_QK_NORM_HEAD && (half == 0 || a.pairing == MRS_SEQ_PAIRS_NEIGHBOURS) && a.dk % 8 == 0 && a.dv % 8 == 0 &&
+      (a.q_ld | a.k_ld | (a.v ? a.v_ld : 0)) % 8 == 0 && al16(a.q) && al16(a.k) && al16(a.v) && al16(a.k_cache) && al16(a.v_cache) &&
+      al16(a.q_norm_w) && al16(a.k_norm_w)) {
+    const int items = (a.heads * a.dk + a.kv_heads * (a.dk + (a.v ? a.dv : 0))) / 8;
+    int th = 64;
+    while (th < 512 && th < items) th *= 2;
+    SEQ_DISPATCH_DTYPE(a.dtype, (attention_prepare_row_kernel<T><<<a.n_tok, th, 0, (cudaStream_t)stream>>>(a)));
+    return launch_status();
+  }
+  if (a.dk % 2 == 0 && a.dv % 2 == 0 && (a.q_ld | a.k_ld | (a.v ? a.v_ld : 0)) % 2 == 0 && al(a.q) && al(a.k) && al(a.v) && al(a.k_cache) && al(a.v_cache) &&
+      (a.pairing == MRS_SEQ_PAIRS_NEIGHBOURS || half % 2 == 0)) {
+    SEQ_DISPATCH_DTYPE(a.dtype, (attention_prepare_vec_kernel<T><<<a.n_tok, warps * 32, bytes, (cudaStream_t)stream>>>(a)));
+    return launch_status();
+  }
   SEQ_DISPATCH_DTYPE(a.dtype, (attention_prepare_kernel<T><<<a.n_tok, warps * 32, bytes, (cudaStream_t)stream>>>(a)));
   return launch_status();
 }
